@@ -390,6 +390,8 @@ int b200_tree_finalize(int depth, int T, const float* pool_scores, const int* po
                        int* fwd_pos, unsigned long long* fwd_mask, int* fwd_prefix, int* tree_position_ids,
                        int* mask_index, int* draft_tokens, int* retrieve, int* tree_info, void* stream);
 int b200_logits_argmax(const void* logits, int R, int V, unsigned long long* best_key, void* stream);
+/* The same for fp32 logits. */
+int b200_logits_argmax_f32(const float* logits, int R, int V, unsigned long long* best_key, void* stream);
 /* Vocabulary-parallel argmax across GPUs: turns the shard-local keys of b200_logits_argmax into global ones
  * (index_offset = first vocabulary row of this GPU's shard) and toggles the top bit so that a signed 64-bit MAX
  * all-reduce orders them; call again with index_offset 0 after the all-reduce to toggle the bit back. */
@@ -400,6 +402,18 @@ int b200_argmax_key_shift(unsigned long long* best_key, int R, unsigned int inde
 int b200_tree_accept(int T, unsigned long long* argmax_key, const int* draft_tokens, const int* retrieve,
                      const int* tree_info, int* ctl, int* y, int* accept_rows, int* out_tokens,
                      int* step_log, void* stream);
+
+/* The same, but a path is accepted over its own nodes only (never over a -1 pad read as node T): for models whose
+ * committed state is advanced over the accepted nodes. */
+int b200_tree_accept_strict(int T, unsigned long long* argmax_key, const int* draft_tokens, const int* retrieve,
+                            const int* tree_info, int* ctl, int* y, int* accept_rows, int* out_tokens,
+                            int* step_log, void* stream);
+/* Decoding without a draft model: the inputs of the next one-row pass (the last token at the committed length), and the
+ * bookkeeping of its greedy token (argmax_key[0] from the argmax of that row). */
+int b200_prep_root(const int* ctl, const int* y, int* fwd_tokens, int* fwd_pos, unsigned long long* fwd_mask,
+                   int* fwd_prefix, void* stream);
+int b200_root_accept(unsigned long long* argmax_key, int* ctl, int* y, int* accept_rows, int* out_tokens, int* step_log,
+                     void* stream);
 
 /* Sampling acceptance at temperature > 0 (no counterpart in the reference, which is greedy only: README.md:9;
  * the same role as evaluate_posterior_greedy + the bookkeeping of generate_step, mlx_eagle.py:311-326,587-599).

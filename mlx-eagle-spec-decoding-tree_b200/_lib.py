@@ -1,6 +1,6 @@
-"""ctypes loader of ``libb200eagle.so``.
+"""ctypes loaders of ``libb200eagle.so`` (``lib()``) and ``libb200hybrid.so`` (``hybrid()``).
 
-There is no fallback: if the library has not been built (``python -m`` of
+There is no fallback: if a library has not been built (``python -m`` of
 ``build.py`` in this directory, or ``__graft_entry__.build()``), importing an
 operator raises.  All tensors handed to the library are CUDA tensors owned by
 torch; the library only sees raw device pointers and the current CUDA stream.
@@ -14,12 +14,14 @@ import torch
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libb200eagle.so")
+HYBRID_LIB_PATH = os.path.join(_HERE, "libb200hybrid.so")
 
 E_NAMES = {-1: "EINVAL (bad shape/size/flags)", -2: "EALIGN (pointer not 16-byte aligned)",
            -3: "EUNSUPPORTED (dtype/group size)", -4: "EWORKSPACE (workspace too small)",
            -5: "ECUDA (CUDA runtime error)", -6: "ELIMIT (size beyond a fixed maximum)"}
 
 _lib = None
+_hybrid = None
 
 
 class B200Error(RuntimeError):
@@ -38,6 +40,35 @@ def lib() -> ctypes.CDLL:
         if os.environ.get("B200_PDL", "1") == "0":
             _lib.b200_set_pdl(0)
     return _lib
+
+
+def hybrid() -> ctypes.CDLL:
+    """The library of the layer-list decoders (``include/b200_hybrid.h``)."""
+    global _hybrid
+    if _hybrid is None:
+        if not os.path.exists(HYBRID_LIB_PATH):
+            raise B200Error(
+                f"{HYBRID_LIB_PATH} is missing: build it first (python {os.path.join(_HERE, 'build.py')}). "
+                "There is no CPU or PyTorch fallback for this path.")
+        l = ctypes.CDLL(HYBRID_LIB_PATH)
+        vp, i32, sz = ctypes.c_void_p, ctypes.c_int, ctypes.c_size_t
+        mp, pp = ctypes.POINTER(HybridModelDesc), ctypes.POINTER(HybridPass)
+        l.b200_hybrid_version.restype = i32
+        l.b200_hybrid_last_cuda_error.restype = i32
+        l.b200_hybrid_set_pdl.restype = None
+        l.b200_hybrid_set_pdl.argtypes = [i32]
+        l.b200_hybrid_attention_workspace_bytes.restype = sz
+        l.b200_hybrid_attention_workspace_bytes.argtypes = [mp, i32]
+        l.b200_hybrid_forward.restype = i32
+        l.b200_hybrid_forward.argtypes = [mp, pp, vp]
+        l.b200_hybrid_commit.restype = i32
+        l.b200_hybrid_commit.argtypes = [mp, vp, i32, vp, vp, i32, vp, i32, vp]
+        l.b200_hybrid_linear.restype = i32
+        l.b200_hybrid_linear.argtypes = [mp, ctypes.POINTER(Linear), vp, i32, i32, vp, i32, i32, vp]
+        if os.environ.get("B200_PDL", "1") == "0":
+            l.b200_hybrid_set_pdl(0)
+        _hybrid = l
+    return _hybrid
 
 
 def _declare(l: ctypes.CDLL) -> None:
@@ -98,6 +129,14 @@ def _declare(l: ctypes.CDLL) -> None:
     l.b200_logits_argmax.argtypes = [vp, i32, i32, vp, vp]
     l.b200_tree_accept.restype = i32
     l.b200_tree_accept.argtypes = [i32] + [vp] * 10
+    l.b200_tree_accept_strict.restype = i32
+    l.b200_tree_accept_strict.argtypes = [i32] + [vp] * 10
+    l.b200_logits_argmax_f32.restype = i32
+    l.b200_logits_argmax_f32.argtypes = [vp, i32, i32, vp, vp]
+    l.b200_prep_root.restype = i32
+    l.b200_prep_root.argtypes = [vp] * 7
+    l.b200_root_accept.restype = i32
+    l.b200_root_accept.argtypes = [vp] * 7
     l.b200_tree_accept_sample_workspace_bytes.restype = sz
     l.b200_tree_accept_sample_workspace_bytes.argtypes = [i32]
     l.b200_tree_accept_sample.restype = i32
@@ -157,11 +196,53 @@ class ForwardDesc(ctypes.Structure):
            ("scales_in_fast_range", ctypes.c_int), ("tp_two_shot", ctypes.c_int), ("requests", ctypes.c_int)])
 
 
+class Linear(ctypes.Structure):
+    """Mirror of ``b200_linear`` (include/b200_hybrid.h)."""
+    _fields_ = [("w", ctypes.c_void_p)] + [(n, ctypes.c_int) for n in ("n", "k", "pitch", "reserved")]
+
+
+class HybridLayer(ctypes.Structure):
+    """Mirror of ``b200_hybrid_layer``."""
+    _fields_ = ([(n, ctypes.c_int) for n in ("mixer", "taps", "heads", "kv_heads", "dim", "vdim", "maps", "window",
+                                             "keep_first", "ff")]
+                + [(n, ctypes.c_float) for n in ("scale", "lambda_", "out_scale")]
+                + [("act", ctypes.c_float * 4), ("reserved", ctypes.c_int)]
+                + [(n, ctypes.c_void_p) for n in ("norm1", "norm2", "conv", "gate_bias", "gate_lower", "head_norm")]
+                + [(n, Linear) for n in ("in_", "out", "up", "down")])
+
+
+class HybridRun(ctypes.Structure):
+    """Mirror of ``b200_hybrid_run``."""
+    _fields_ = ([("layer", ctypes.c_int), ("inject", ctypes.c_int)]
+                + [(n, ctypes.c_longlong) for n in ("conv_off", "k_off", "v_off", "state_off", "pend_h", "pend_g", "pend_v")])
+
+
+class HybridModelDesc(ctypes.Structure):
+    """Mirror of ``b200_hybrid_model``."""
+    _fields_ = ([(n, ctypes.c_int) for n in ("act_type", "width", "vocab", "n_layers", "n_runs", "max_rows", "injects",
+                                             "conv_max_taps")]
+                + [(n, ctypes.c_float) for n in ("eps", "residual_mult", "softcap")] + [("reserved", ctypes.c_int)]
+                + [(n, ctypes.c_void_p) for n in ("embed", "final_norm")]
+                + [("layers", ctypes.POINTER(HybridLayer)), ("runs", ctypes.POINTER(HybridRun))]
+                + [(n, ctypes.c_void_p) for n in ("dev_layers", "dev_runs")] + [("head", Linear)]
+                + [(n, ctypes.c_void_p) for n in ("x", "emb", "hb", "qb", "gb", "vb", "gf", "o32", "ab", "zb", "zab",
+                                                  "pending", "attn_part")]
+                + [("attn_part_bytes", ctypes.c_size_t), ("error", ctypes.c_void_p)])
+
+
+class HybridPass(ctypes.Structure):
+    """Mirror of ``b200_hybrid_pass``."""
+    _fields_ = ([(n, ctypes.c_int) for n in ("M", "tree", "write_off", "tail", "rows_out", "cache_rows", "max_keys", "reserved")]
+                + [(n, ctypes.c_void_p) for n in ("tokens", "pos", "mask", "prefix", "out_rows", "row_index", "tail_pos", "cache",
+                                                  "logits", "logits16", "dump")])
+
+
 def check(rc: int, what: str) -> None:
     if rc != 0:
         extra = ""
         if rc == -5:
-            extra = f" (cudaError {lib().b200_last_cuda_error()})"
+            l = hybrid() if what.startswith("b200_hybrid") else lib()
+            extra = f" (cudaError {l.b200_hybrid_last_cuda_error() if l is _hybrid else l.b200_last_cuda_error()})"
         raise B200Error(f"{what} failed: {E_NAMES.get(rc, rc)}{extra}")
 
 

@@ -1,0 +1,296 @@
+// Gated linear recurrence of the hybrid decoders (the forget gate also decides what is written):
+//     S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T   computed as   S += (1 - f) (v - S),      o_t = S_t^T q_t,
+// all in fp32, the state [heads][dim][vdim] carried in the request's cache.
+//
+//   scan_kernel    chain passes, any number of rows: CTA = (head, 32 state columns), warp = a slice of the state's rows,
+//                  lane = column; the slice lives in registers, tokens come in blocks through shared memory, the warps'
+//                  parts of an output are added once per block.  The new state is written back.
+//   tree_kernel    tree passes: nothing may change the state yet.  Row m's output is written out along its path:
+//                  o = S_0^T (q prod f) + sum over the path's rows a of (q . (1 - f_a) prod of the later f) v_a.
+//   commit_kernel  advances convolution inputs, states and K/V rows over accepted rows, for every layer run at once.
+//   head_norm      per-head RMS norm of the outputs with the head weight, to the activation type.
+#include "hybrid.cuh"
+
+namespace b200 {
+namespace hybrid {
+namespace {
+
+constexpr int kWarps = 8;
+constexpr int kMaxDim = 256;
+
+template <typename T, int DR, int TB>    // state rows of a warp, tokens of a block
+__global__ void __launch_bounds__(kWarps * 32) scan_kernel(const T* __restrict__ q, const float* __restrict__ gf, const T* __restrict__ v,
+                                                           float* __restrict__ state, float* __restrict__ o, int M, int H, int d, int dv) {
+    pdl_wait();
+    pdl_launch_dependents();
+    constexpr int D = kWarps * DR;
+    constexpr int PER = TB * D / (kWarps * 32), PERV = (TB * 32 + kWarps * 32 - 1) / (kWarps * 32);
+    __shared__ __align__(16) float sg[TB][D];
+    __shared__ __align__(16) float sq[TB][D];
+    __shared__ float sv[TB][32];
+    __shared__ float part[kWarps][TB][32];
+    const int h = blockIdx.y, c0 = blockIdx.x * 32, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int col = c0 + lane;
+    float S[DR];
+    float* sbase = state + ((size_t)h * d + warp * DR) * dv + col;
+#pragma unroll
+    for (int r = 0; r < DR; r++) S[r] = (warp * DR + r < d && col < dv) ? sbase[(size_t)r * dv] : 0.f;
+    float pg[PER], pq[PER], pv[PERV];
+    auto fetch = [&](int t0) {
+#pragma unroll
+        for (int i = 0; i < PER; i++) {
+            const int e = tid + i * kWarps * 32, t = e / D, c = e % D;
+            const bool in = t0 + t < M && c < d;
+            pg[i] = in ? gf[((size_t)(t0 + t) * H + h) * d + c] : 0.f;
+            pq[i] = in ? to_f32<T>(q[((size_t)(t0 + t) * H + h) * d + c]) : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < PERV; i++) {
+            const int e = tid + i * kWarps * 32, t = e / 32, c = c0 + (e & 31);
+            pv[i] = (t < TB && t0 + t < M && c < dv) ? to_f32<T>(v[((size_t)(t0 + t) * H + h) * dv + c]) : 0.f;
+        }
+    };
+    fetch(0);
+    for (int t0 = 0; t0 < M; t0 += TB) {
+        __syncthreads();                               // the previous block's parts have been read
+#pragma unroll
+        for (int i = 0; i < PER; i++) {
+            const int e = tid + i * kWarps * 32;
+            (&sg[0][0])[e] = pg[i];
+            (&sq[0][0])[e] = pq[i];
+        }
+#pragma unroll
+        for (int i = 0; i < PERV; i++) {
+            const int e = tid + i * kWarps * 32;
+            if (e < TB * 32) (&sv[0][0])[e] = pv[i];
+        }
+        __syncthreads();
+        if (t0 + TB < M) fetch(t0 + TB);
+        const int nt = min(TB, M - t0);
+#pragma unroll 2
+        for (int t = 0; t < nt; t++) {
+            const float vt = sv[t][lane];
+            float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+            for (int r = 0; r < DR; r += 4) {
+                const float4 g4 = *reinterpret_cast<const float4*>(&sg[t][warp * DR + r]);
+                const float4 q4 = *reinterpret_cast<const float4*>(&sq[t][warp * DR + r]);
+                S[r] = fmaf(g4.x, vt - S[r], S[r]);
+                S[r + 1] = fmaf(g4.y, vt - S[r + 1], S[r + 1]);
+                S[r + 2] = fmaf(g4.z, vt - S[r + 2], S[r + 2]);
+                S[r + 3] = fmaf(g4.w, vt - S[r + 3], S[r + 3]);
+                a0 = fmaf(q4.x, S[r], a0);
+                a1 = fmaf(q4.y, S[r + 1], a1);
+                a0 = fmaf(q4.z, S[r + 2], a0);
+                a1 = fmaf(q4.w, S[r + 3], a1);
+            }
+            part[warp][t][lane] = a0 + a1;
+        }
+        __syncthreads();
+        for (int e = tid; e < nt * 32; e += kWarps * 32) {
+            const int t = e >> 5, c = e & 31;
+            float a = 0.f;
+#pragma unroll
+            for (int w = 0; w < kWarps; w++) a += part[w][t][c];
+            if (c0 + c < dv) o[((size_t)(t0 + t) * H + h) * dv + c0 + c] = a;
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < DR; r++)
+        if (warp * DR + r < d && col < dv) sbase[(size_t)r * dv] = S[r];
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) tree_kernel(const T* __restrict__ q, const float* __restrict__ pend_g, const T* __restrict__ pend_v,
+                                                   const float* __restrict__ state, const unsigned long long* __restrict__ mask,
+                                                   float* __restrict__ o, int H, int d, int dv) {
+    pdl_wait();
+    pdl_launch_dependents();
+    __shared__ float sw[B200_HYBRID_PENDING][4];
+    __shared__ float sqs[kMaxDim];
+    const int h = blockIdx.x, m = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const unsigned long long path = mask[m];             // the row itself and its ancestors among the tail rows
+    float qi[2], suf[2];
+#pragma unroll
+    for (int k = 0; k < 2; k++) {
+        const int i = tid + 128 * k;
+        qi[k] = i < d ? to_f32<T>(q[((size_t)m * H + h) * d + i]) : 0.f;
+        suf[k] = 1.f;
+    }
+    for (unsigned long long left = path; left != 0ull;) {   // newest row first
+        const int a = 63 - __clzll((long long)left);
+        left &= ~(1ull << a);
+        float c = 0.f;
+#pragma unroll
+        for (int k = 0; k < 2; k++) {
+            const int i = tid + 128 * k;
+            if (i < d) {
+                const float g = pend_g[((size_t)a * H + h) * d + i];
+                c = fmaf(qi[k] * suf[k], g, c);
+                suf[k] *= 1.f - g;
+            }
+        }
+        c = warp_sum(c);
+        if (lane == 0) sw[a][warp] = c;
+    }
+#pragma unroll
+    for (int k = 0; k < 2; k++)
+        if (tid + 128 * k < d) sqs[tid + 128 * k] = qi[k] * suf[k];
+    __syncthreads();
+    for (int c = tid; c < dv; c += 128) {
+        float acc = 0.f;
+        const float* s = state + (size_t)h * d * dv + c;
+#pragma unroll 8
+        for (int i = 0; i < d; i++) acc = fmaf(sqs[i], s[(size_t)i * dv], acc);
+        for (unsigned long long left = path; left != 0ull; left &= left - 1ull) {
+            const int a = __ffsll((long long)left) - 1;
+            acc = fmaf(sw[a][0] + sw[a][1] + sw[a][2] + sw[a][3], to_f32<T>(pend_v[((size_t)a * H + h) * dv + c]), acc);
+        }
+        o[((size_t)m * H + h) * dv + c] = acc;
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) head_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, T* __restrict__ out, int M, int H,
+                                                        int dv, int pitch, float eps) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int unit = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (unit >= M * H) return;
+    const int m = unit / H, h = unit - m * H;
+    const float* row = o + (size_t)unit * dv;
+    float ss = 0.f;
+    for (int c = lane; c < dv; c += 32) { const float x = row[c]; ss = fmaf(x, x, ss); }
+    const float rstd = rsqrtf(warp_sum(ss) / (float)dv + eps);
+    T* dst = out + (size_t)m * pitch + (size_t)h * dv;
+    for (int c = lane; c < dv; c += 32) dst[c] = from_f32<T>(row[c] * rstd * w[c]);
+}
+
+struct CommitParams {
+    const b200_hybrid_layer* layers;
+    const b200_hybrid_run* runs;
+    char* cache;
+    char* pending;
+    const int* count;
+    const int* rows;
+    const int* prefix;
+    int width, cap, fixed_count, tree_rows, states, compact;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) commit_kernel(const CommitParams p) {
+    pdl_wait();
+    pdl_launch_dependents();
+    __shared__ int srow[B200_HYBRID_PENDING];
+    const b200_hybrid_run& r = p.runs[blockIdx.x];
+    const b200_hybrid_layer& l = p.layers[r.layer];
+    int n = p.fixed_count > 0 ? p.fixed_count : p.count[0] + 1;
+    n = min(max(n, 0), B200_HYBRID_PENDING);
+    for (int i = threadIdx.x; i < n; i += 256) {
+        int s = (i == 0 || p.rows == nullptr || p.fixed_count > 0) ? i : p.rows[i];
+        if (s < 0) s += p.tree_rows;
+        srow[i] = min(max(s, 0), B200_HYBRID_PENDING - 1);
+    }
+    __syncthreads();
+    const int first = blockIdx.y * 256 + threadIdx.x, step = gridDim.y * 256;
+    const int prev = l.taps - 1;
+    if (prev > 0) {
+        float* state = reinterpret_cast<float*>(p.cache + r.conv_off);
+        const float* pend = reinterpret_cast<const float*>(p.pending + r.pend_h);
+        for (int c = first; c < p.width; c += step) {
+            float nv[B200_HYBRID_MAX_TAPS];
+#pragma unroll
+            for (int j = 0; j < B200_HYBRID_MAX_TAPS; j++) {
+                const int i = n - prev + j;
+                nv[j] = 0.f;
+                if (j < prev) nv[j] = i >= 0 ? pend[(size_t)srow[i] * p.width + c] : state[(size_t)(i + prev) * p.width + c];
+            }
+#pragma unroll
+            for (int j = 0; j < B200_HYBRID_MAX_TAPS; j++)
+                if (j < prev) state[(size_t)j * p.width + c] = nv[j];
+        }
+    }
+    if (p.states && l.mixer == B200_MIXER_RECURRENCE) {
+        float* state = reinterpret_cast<float*>(p.cache + r.state_off);
+        const float* pg = reinterpret_cast<const float*>(p.pending + r.pend_g);
+        const T* pv = reinterpret_cast<const T*>(p.pending + r.pend_v);
+        const int per = l.dim * l.vdim, total = l.heads * per;
+        for (int e = first; e < total; e += step) {
+            const int h = e / per, x = e - h * per, i = x / l.vdim, c = x - i * l.vdim;
+            float s = state[e];
+            for (int t = 0; t < n; t++) {
+                const float g = pg[((size_t)srow[t] * l.heads + h) * l.dim + i];
+                const float v = to_f32<T>(pv[((size_t)srow[t] * l.heads + h) * l.vdim + c]);
+                s = fmaf(g, v - s, s);
+            }
+            state[e] = s;
+        }
+    }
+    if (p.compact && l.mixer == B200_MIXER_ATTENTION) {
+        const int P = p.prefix[0];
+        const int ke = l.maps * round_up(l.dim, 16), ve = round_up(l.vdim, 16), per = ke + ve;
+        for (int e = first; e < l.kv_heads * per; e += step) {
+            const int g = e / per, x = e - g * per;
+            T* base = x < ke ? reinterpret_cast<T*>(p.cache + r.k_off) + (size_t)g * p.cap * ke + x
+                             : reinterpret_cast<T*>(p.cache + r.v_off) + (size_t)g * p.cap * ve + (x - ke);
+            const int pitch = x < ke ? ke : ve;
+            // rows ascend along a path, so no source is overwritten before it is read
+            for (int i = 1; i < n; i++)
+                if (srow[i] != i && P + srow[i] < p.cap) base[(size_t)(P + i) * pitch] = base[(size_t)(P + srow[i]) * pitch];
+        }
+    }
+}
+
+template <typename T>
+int launch_scan(const b200_hybrid_model& m, const b200_hybrid_layer& l, float* state, int M, cudaStream_t st) {
+    const dim3 grid((l.vdim + 31) / 32, l.heads), block(kWarps * 32);
+    const T* q = static_cast<const T*>(m.qb);
+    const T* v = static_cast<const T*>(m.vb);
+    if (l.dim <= 32) launch_kernel(scan_kernel<T, 4, 16>, grid, block, 0, st, q, m.gf, v, state, m.o32, M, l.heads, l.dim, l.vdim);
+    else if (l.dim <= 64) launch_kernel(scan_kernel<T, 8, 16>, grid, block, 0, st, q, m.gf, v, state, m.o32, M, l.heads, l.dim, l.vdim);
+    else if (l.dim <= 128) launch_kernel(scan_kernel<T, 16, 16>, grid, block, 0, st, q, m.gf, v, state, m.o32, M, l.heads, l.dim, l.vdim);
+    else launch_kernel(scan_kernel<T, 32, 8>, grid, block, 0, st, q, m.gf, v, state, m.o32, M, l.heads, l.dim, l.vdim);
+    return check_launch();
+}
+
+template <typename T>
+int recurrence(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_run& r, const b200_hybrid_pass& p, cudaStream_t st) {
+    float* state = reinterpret_cast<float*>(static_cast<char*>(p.cache) + r.state_off);
+    int rc;
+    if (p.tree) {
+        launch_kernel(tree_kernel<T>, dim3(l.heads, p.M), dim3(128), 0, st, static_cast<const T*>(m.qb),
+                      reinterpret_cast<const float*>(static_cast<const char*>(m.pending) + r.pend_g),
+                      reinterpret_cast<const T*>(static_cast<const char*>(m.pending) + r.pend_v), static_cast<const float*>(state), p.mask,
+                      m.o32, l.heads, l.dim, l.vdim);
+        rc = check_launch();
+    } else {
+        rc = launch_scan<T>(m, l, state, p.M, st);
+    }
+    if (rc != B200_OK) return rc;
+    launch_kernel(head_norm_kernel<T>, dim3((p.M * l.heads + 3) / 4), dim3(128), 0, st, static_cast<const float*>(m.o32), l.head_norm,
+                  static_cast<T*>(m.ab), p.M, l.heads, l.vdim, round_up(l.heads * l.vdim, 64), m.eps);
+    return check_launch();
+}
+
+}  // namespace
+
+int launch_recurrence(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_run& r, const b200_hybrid_pass& p,
+                      cudaStream_t st) {
+    if (l.dim > kMaxDim) return B200_ELIMIT;
+    return m.act_type == B200_ACT_F32 ? recurrence<float>(m, l, r, p, st) : recurrence<bf16>(m, l, r, p, st);
+}
+
+int launch_commit(const b200_hybrid_model& m, void* cache, int cache_rows, int fixed_count, const int* count, const int* rows, int tree_rows,
+                  const int* prefix, int states, int compact, cudaStream_t st) {
+    CommitParams p{};
+    p.layers = m.dev_layers; p.runs = m.dev_runs; p.cache = static_cast<char*>(cache); p.pending = static_cast<char*>(m.pending);
+    p.count = count; p.rows = rows; p.prefix = prefix; p.width = m.width; p.cap = cache_rows; p.fixed_count = fixed_count;
+    p.tree_rows = tree_rows; p.states = states; p.compact = compact;
+    const dim3 grid(m.n_runs, states ? 32 : 4);
+    if (m.act_type == B200_ACT_F32) launch_kernel(commit_kernel<float>, grid, dim3(256), 0, st, p);
+    else launch_kernel(commit_kernel<bf16>, grid, dim3(256), 0, st, p);
+    return check_launch();
+}
+
+}  // namespace hybrid
+}  // namespace b200

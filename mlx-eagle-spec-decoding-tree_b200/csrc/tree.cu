@@ -187,15 +187,19 @@ __global__ void __launch_bounds__(256) row_topk_kernel(const __half* __restrict_
     }
 }
 
-__global__ void row_argmax_kernel(const __half* __restrict__ logits, int V, unsigned long long* __restrict__ best_key) {
+__device__ __forceinline__ float logit_f32(__half v) { return __half2float(v); }
+__device__ __forceinline__ float logit_f32(float v) { return v; }
+
+template <typename L>
+__global__ void row_argmax_kernel(const L* __restrict__ logits, int V, unsigned long long* __restrict__ best_key) {
     pdl_wait();
     pdl_launch_dependents();
     const int r = blockIdx.y;
     const int begin = blockIdx.x * kTopkChunk, end = min(V, begin + kTopkChunk);
-    const __half* row = logits + (size_t)r * V;
+    const L* row = logits + (size_t)r * V;
     unsigned long long best = 0;
     for (int i = begin + threadIdx.x; i < end; i += blockDim.x) {
-        const unsigned long long k = make_key(__half2float(row[i]), (uint32_t)i);
+        const unsigned long long k = make_key(logit_f32(row[i]), (uint32_t)i);
         best = k > best ? k : best;
     }
     best = warp_max_key(best);
@@ -501,6 +505,7 @@ __device__ void commit_step(int* ctl, int* y, int* out_tokens, int* step_log, in
 // ---------------------------------------------------------------- greedy acceptance (1 warp)
 struct AcceptParams {
     int T;
+    int strict;                          // a path ends at its leaf (else a -1 pad stands for node T, as in the reference)
     unsigned long long* argmax_key;      // [T+1] (cleared on exit)
     const int* draft_tokens;             // [T+1]
     const int* retrieve;                 // [T][kMaxDepth+2]
@@ -529,7 +534,7 @@ __global__ void tree_accept_kernel(const AcceptParams p) {
             a = a < 0 ? a + T + 1 : a;
             b = b < 0 ? b + T + 1 : b;
             const int pred = (int)key_index(p.argmax_key[a]);
-            alive = alive && (p.draft_tokens[b] == pred);
+            alive = alive && (p.draft_tokens[b] == pred) && (!p.strict || p.retrieve[lane * RW + j + 1] >= 0);
             len += alive ? 1 : 0;
         }
     }
@@ -557,6 +562,29 @@ __global__ void tree_accept_kernel(const AcceptParams p) {
     }
     __syncwarp();
     if (lane <= T) p.argmax_key[lane] = 0ull;
+}
+
+// ---------------------------------------------------------------- decoding without a draft (a tree of the root alone)
+__global__ void prep_root_kernel(const int* __restrict__ ctl, const int* __restrict__ y, int* fwd_tokens, int* fwd_pos,
+                                 unsigned long long* fwd_mask, int* fwd_prefix) {
+    pdl_wait();
+    pdl_launch_dependents();
+    if (threadIdx.x != 0) return;
+    const int P = ctl[CTL_BASE_LEN];
+    fwd_tokens[0] = y[ctl[CTL_ACCEPT]];
+    fwd_pos[0] = P;
+    fwd_mask[0] = 1ull;
+    fwd_prefix[0] = P;
+}
+
+__global__ void root_accept_kernel(unsigned long long* argmax_key, int* ctl, int* y, int* accept_rows, int* out_tokens, int* step_log) {
+    pdl_wait();
+    pdl_launch_dependents();
+    if (threadIdx.x != 0) return;
+    accept_rows[0] = 0;
+    for (int j = 0; j < kK; j++) y[j] = 0;
+    commit_step(ctl, y, out_tokens, step_log, 0, 0, (int)key_index(argmax_key[0]));
+    argmax_key[0] = 0ull;
 }
 
 // ---------------------------------------------------------------- sampling acceptance
@@ -867,7 +895,15 @@ int b200_tree_finalize(int depth, int T, const float* pool_scores, const int* po
 int b200_logits_argmax(const void* logits, int R, int V, unsigned long long* best_key, void* stream) {
     if (!logits || !best_key || R < 1 || R > 32 || V < 1) return B200_EINVAL;
     dim3 grid(b200::nblk_for(V), R);
-    b200::launch_kernel(b200::row_argmax_kernel, dim3(grid), dim3(256), 0, static_cast<cudaStream_t>(stream), static_cast<const __half*>(logits), V, best_key);
+    b200::launch_kernel(b200::row_argmax_kernel<__half>, dim3(grid), dim3(256), 0, static_cast<cudaStream_t>(stream), static_cast<const __half*>(logits), V, best_key);
+    return b200::check_launch();
+}
+
+// The same for fp32 logits.
+int b200_logits_argmax_f32(const float* logits, int R, int V, unsigned long long* best_key, void* stream) {
+    if (!logits || !best_key || R < 1 || R > 32 || V < 1) return B200_EINVAL;
+    b200::launch_kernel(b200::row_argmax_kernel<float>, dim3(b200::nblk_for(V), R), dim3(256), 0, static_cast<cudaStream_t>(stream),
+                        logits, V, best_key);
     return b200::check_launch();
 }
 
@@ -882,17 +918,46 @@ int b200_argmax_key_shift(unsigned long long* best_key, int R, unsigned int inde
 }
 
 // evaluate_posterior_greedy + the bookkeeping of generate_step (mlx_eagle.py:311-326,582-599).
-int b200_tree_accept(int T, unsigned long long* argmax_key, const int* draft_tokens, const int* retrieve,
-                     const int* tree_info, int* ctl, int* y, int* accept_rows, int* out_tokens,
-                     int* step_log, void* stream) {
+static int launch_accept(int T, int strict, unsigned long long* argmax_key, const int* draft_tokens, const int* retrieve,
+                         const int* tree_info, int* ctl, int* y, int* accept_rows, int* out_tokens, int* step_log, void* stream) {
     if (T < 1 || T > 31 || !argmax_key || !draft_tokens || !retrieve || !tree_info || !ctl || !y ||
         !accept_rows || !out_tokens || !step_log)
         return B200_EINVAL;
     b200::AcceptParams p{};
-    p.T = T; p.argmax_key = argmax_key; p.draft_tokens = draft_tokens; p.retrieve = retrieve;
+    p.T = T; p.strict = strict; p.argmax_key = argmax_key; p.draft_tokens = draft_tokens; p.retrieve = retrieve;
     p.tree_info = tree_info; p.ctl = ctl; p.y = y; p.accept_rows = accept_rows; p.out_tokens = out_tokens;
     p.step_log = step_log;
     b200::launch_kernel(b200::tree_accept_kernel, dim3(1), dim3(32), 0, static_cast<cudaStream_t>(stream), p);
+    return b200::check_launch();
+}
+
+int b200_tree_accept(int T, unsigned long long* argmax_key, const int* draft_tokens, const int* retrieve,
+                     const int* tree_info, int* ctl, int* y, int* accept_rows, int* out_tokens,
+                     int* step_log, void* stream) {
+    return launch_accept(T, 0, argmax_key, draft_tokens, retrieve, tree_info, ctl, y, accept_rows, out_tokens, step_log, stream);
+}
+
+// The same, but a path is accepted over its own nodes only: what models need whose committed state is rebuilt from
+// the accepted nodes.
+int b200_tree_accept_strict(int T, unsigned long long* argmax_key, const int* draft_tokens, const int* retrieve,
+                            const int* tree_info, int* ctl, int* y, int* accept_rows, int* out_tokens,
+                            int* step_log, void* stream) {
+    return launch_accept(T, 1, argmax_key, draft_tokens, retrieve, tree_info, ctl, y, accept_rows, out_tokens, step_log, stream);
+}
+
+// Decoding without a draft: the inputs of the next one-row pass, and its bookkeeping.
+int b200_prep_root(const int* ctl, const int* y, int* fwd_tokens, int* fwd_pos, unsigned long long* fwd_mask, int* fwd_prefix,
+                   void* stream) {
+    if (!ctl || !y || !fwd_tokens || !fwd_pos || !fwd_mask || !fwd_prefix) return B200_EINVAL;
+    b200::launch_kernel(b200::prep_root_kernel, dim3(1), dim3(32), 0, static_cast<cudaStream_t>(stream), ctl, y, fwd_tokens, fwd_pos,
+                        fwd_mask, fwd_prefix);
+    return b200::check_launch();
+}
+
+int b200_root_accept(unsigned long long* argmax_key, int* ctl, int* y, int* accept_rows, int* out_tokens, int* step_log, void* stream) {
+    if (!argmax_key || !ctl || !y || !accept_rows || !out_tokens || !step_log) return B200_EINVAL;
+    b200::launch_kernel(b200::root_accept_kernel, dim3(1), dim3(32), 0, static_cast<cudaStream_t>(stream), argmax_key, ctl, y, accept_rows,
+                        out_tokens, step_log);
     return b200::check_launch();
 }
 
@@ -905,7 +970,7 @@ int b200_tree_accept_sample(int T, int V, const void* logits, uint32_t* row_max,
                             const int* draft_tokens, const int* mask_index, double temperature, int* ctl, int* y,
                             int* accept_rows, int* out_tokens, int* step_log, void* workspace, size_t workspace_bytes,
                             void* stream) {
-    if (T < 1 || T > 31 || V < 1 || !logits || !row_max || !row_sum || !draft_tokens || !mask_index || !ctl || !y ||
+    if (T < 0 || T > 31 || V < 1 || !logits || !row_max || !row_sum || !draft_tokens || !mask_index || !ctl || !y ||
         !accept_rows || !out_tokens || !step_log || !workspace || !(temperature > 0.0))
         return B200_EINVAL;
     if (workspace_bytes < b200_tree_accept_sample_workspace_bytes(V)) return B200_EWORKSPACE;

@@ -36,7 +36,7 @@ CTL_LOG_CAP, CTL_EOS, CTL_DONE, CTL_STOP_N, CTL_SEED, CTL_DRAW = 8, 9, 10, 11, 1
 class SpecDecoder:
     """Device-resident state and launch sequence of the speculative decoding loop."""
 
-    def __init__(self, base_model: Model, draft_model: Model, depth: int, verify_num_tokens: int,
+    def __init__(self, base_model: Model, draft_model: Optional[Model], depth: int, verify_num_tokens: int,
                  cache_rows: int, max_out_tokens: int = 4096, max_steps: int = 4096, k: int = K,
                  base_cache: Optional[KVCache] = None, draft_cache: Optional[KVCache] = None, req: int = 0,
                  temperature: float = 0.0, seed: int = 0):
@@ -45,7 +45,9 @@ class SpecDecoder:
         if not (0 <= depth <= 6):
             raise _lib.B200Error("depth must be in 0..6 (accepted tokens + 1 must fit the 8-row catch-up pass)")
         T = verify_num_tokens
-        if not (1 <= T <= 31) or T > K + K * K * depth:
+        if draft_model is None:                   # no draft: a step is one target pass on the last token
+            depth, T = 0, 0
+        elif not (1 <= T <= 31) or T > K + K * K * depth:
             raise _lib.B200Error("verify_num_tokens must be <= 31 and <= pool size (README: 7, 15, 23 or 31)")
         self.base, self.draft = base_model, draft_model
         self.depth, self.T = depth, T
@@ -58,7 +60,9 @@ class SpecDecoder:
         self.device = dev
         # (a request of a BatchSpecDecoder gets its slabs of the shared caches and its row group ``req``)
         self.base_cache = base_cache if base_cache is not None else base_model.make_cache(cache_rows)
-        self.draft_cache = draft_cache if draft_cache is not None else draft_model.make_cache(cache_rows)
+        if draft_cache is None and draft_model is not None:
+            draft_cache = draft_model.make_cache(cache_rows)
+        self.draft_cache = draft_cache
         self.req = req
         i32 = dict(dtype=torch.int32, device=dev)
         i64 = dict(dtype=torch.int64, device=dev)
@@ -73,7 +77,7 @@ class SpecDecoder:
         self.topk_cs_index = torch.zeros(K, **i32)
         self.row_max = torch.zeros(MAX_ROWS, **i32)
         self.row_sum = torch.zeros(MAX_ROWS, **i64)
-        nblk = _lib.lib().b200_topk_blocks(draft_model.args.vocab_size)
+        nblk = _lib.lib().b200_topk_blocks(draft_model.args.vocab_size) if draft_model is not None else 1
         self.cand = torch.zeros(K * nblk * K, **i64)
         self.argmax_key = torch.zeros(MAX_ROWS, **i64)
         self.tree_position_ids = torch.zeros(MAX_ROWS, **i32)
@@ -89,9 +93,11 @@ class SpecDecoder:
         self.max_steps = max_steps
         self.graph: Optional[torch.cuda.CUDAGraph] = None
         self.base_logits = None
-        self.kernel_launches_per_step = (
-            (depth + 1) * draft_model.launches_per_forward + base_model.launches_per_forward
-            + 1 + (depth + 1) * 4 + 1 + 1 + 1 + 1)
+        self.kernel_launches_per_step = base_model.launches_per_forward + 3      # ... + input, argmax, acceptance
+        if draft_model is not None:
+            self.kernel_launches_per_step = (
+                (depth + 1) * draft_model.launches_per_forward + base_model.launches_per_forward
+                + 1 + (depth + 1) * 4 + 1 + 1 + 1 + 1)
         if base_model.tp is not None:                    # argmax combine over peer memory, or two key shifts around NCCL
             self.kernel_launches_per_step += 1 if base_model.tp.peers is not None else 2
 
@@ -104,9 +110,10 @@ class SpecDecoder:
         need = n + 8 * (self.depth + 1) + 40
         if need > self.base_cache.rows:
             raise _lib.B200Error(f"cache of {self.base_cache.rows} rows cannot hold a {n}-token prompt")
-        self.base_cache.offset = 0
-        self.draft_cache.offset = 0
-        self.draft(prompt[None], cache=self.draft_cache, logits_last_only=True)
+        self.base_cache.reset()
+        if self.draft is not None:
+            self.draft_cache.reset()
+            self.draft(prompt[None], cache=self.draft_cache, logits_last_only=True)
         logits = self.base(prompt[None], cache=self.base_cache, logits_last_only=True)
         draws = 0
         if self.temperature > 0.0:
@@ -114,7 +121,7 @@ class SpecDecoder:
             self.row_max.zero_()
             self.row_sum.zero_()
             tok = torch.zeros(1, dtype=torch.int32, device=self.device)
-            row = logits[0, -1].contiguous()
+            row = logits[0, -1].half().contiguous()
             _lib.check(_lib.lib().b200_sample_token(
                 _lib.ptr(row), self.base.args.vocab_size, self.temperature, self.seed & 0xFFFFFFFF, 0,
                 _lib.ptr(self.row_max), _lib.ptr(self.row_sum), _lib.ptr(self.sample_ws), self.sample_ws.numel(),
@@ -161,6 +168,7 @@ class SpecDecoder:
         V = d.args.vocab_size
         self._prep_catchup()
         logits = d.forward_device(K, self.draft_cache, 0, K, logits_rows=1, row_index=self.sel_row)
+        d.commit_catchup(self.draft_cache, self.ctl[CTL_ACCEPT:])
         self._expand(logits, 1, V, -1, st)
         for i in range(self.depth):
             logits = d.forward_device(K, self.draft_cache, K * i, K * (i + 1))
@@ -199,6 +207,14 @@ class SpecDecoder:
         self._draft_tree()
         self._finalize()
 
+    def _root_pass(self):
+        """Without a draft: one target pass on the last token."""
+        L, p, ck = _lib.lib(), _lib.ptr, _lib.check
+        tok, pos, mask, prefix = self._inputs(self.base.fwd, 1)
+        ck(L.b200_prep_root(p(self.ctl), p(self.y), p(tok), p(pos), p(mask), p(prefix), _lib.stream_ptr(self.device)), "b200_prep_root")
+        kw = dict(commit=True) if self.base.stateful else {}        # the row is part of the sequence in any case
+        self.base_logits = self.base.forward_device(1, self.base_cache, 0, 1, **kw)
+
     def _accept(self):
         L, p, ck = _lib.lib(), _lib.ptr, _lib.check
         st = _lib.stream_ptr(self.device)
@@ -209,12 +225,10 @@ class SpecDecoder:
                                          p(self.draft_tokens), p(self.mask_index), self.temperature, p(self.ctl), p(self.y),
                                          p(self.accept_rows), p(self.out_tokens), p(self.step_log), p(self.sample_ws),
                                          self.sample_ws.numel(), st), "b200_tree_accept_sample")
-            ck(L.b200_kv_compact(p(self.base_cache.data), a.num_hidden_layers, a.num_key_value_heads,
-                                 self.base_cache.rows, a.head_dim, p(self.accept_rows), p(self.ctl), st),
-               "b200_kv_compact")
+            if self.draft is not None:
+                base.commit_accepted(self.base_cache, self.accept_rows, self.ctl, self.T + 1)
             return
-        ck(L.b200_logits_argmax(p(self.base_logits), self.T + 1, base.vocab_local, p(self.argmax_key), st),
-           "b200_logits_argmax")
+        base.argmax_rows(self.base_logits, self.T + 1, self.argmax_key)
         if base.tp is not None and base.tp.peers is not None:
             # vocabulary-parallel head: every shard's per-node (max, argmax) keys, combined over peer memory
             tp = base.tp
@@ -225,17 +239,23 @@ class SpecDecoder:
             ck(L.b200_argmax_key_shift(p(self.argmax_key), self.T + 1, base.vocab_offset, st), "b200_argmax_key_shift")
             base.tp.all_reduce_max(self.argmax_key[: self.T + 1])
             ck(L.b200_argmax_key_shift(p(self.argmax_key), self.T + 1, 0, st), "b200_argmax_key_shift")
-        ck(L.b200_tree_accept(self.T, p(self.argmax_key), p(self.draft_tokens), p(self.retrieve), p(self.tree_info),
-                              p(self.ctl), p(self.y), p(self.accept_rows), p(self.out_tokens), p(self.step_log), st),
+        if self.draft is None:
+            ck(L.b200_root_accept(p(self.argmax_key), p(self.ctl), p(self.y), p(self.accept_rows), p(self.out_tokens),
+                                  p(self.step_log), st), "b200_root_accept")
+            return
+        accept = L.b200_tree_accept_strict if base.stateful else L.b200_tree_accept
+        ck(accept(self.T, p(self.argmax_key), p(self.draft_tokens), p(self.retrieve), p(self.tree_info),
+                  p(self.ctl), p(self.y), p(self.accept_rows), p(self.out_tokens), p(self.step_log), st),
            "b200_tree_accept")
-        ck(L.b200_kv_compact(p(self.base_cache.data), a.num_hidden_layers, a.num_key_value_heads,
-                             self.base_cache.rows, a.head_dim, p(self.accept_rows), p(self.ctl), st),
-           "b200_kv_compact")
+        base.commit_accepted(self.base_cache, self.accept_rows, self.ctl, self.T + 1)
 
     def step(self):
-        """Launch one whole speculative step (no host synchronisation)."""
-        self._draft_tree()
-        self._finalize_and_verify()
+        """Launch one whole speculative step (no host synchronisation); without a draft, one plain decoding step."""
+        if self.draft is None:
+            self._root_pass()
+        else:
+            self._draft_tree()
+            self._finalize_and_verify()
         self._accept()
 
     def capture(self):
@@ -258,7 +278,7 @@ class SpecDecoder:
         """One eager step on a dummy prompt (sets kernel attributes, sizes workspaces), then the graph
         capture.  Call once after construction; ``generate`` then only replays."""
         g = torch.Generator().manual_seed(0)
-        v = min(self.base.args.vocab_size, self.draft.args.vocab_size)
+        v = min(m.args.vocab_size for m in (self.base, self.draft) if m is not None)
         self.prefill(torch.randint(0, v, (8,), generator=g, dtype=torch.int32))
         self.step()
         if capture and (self.base.tp is None or self.base.can_fuse()):
@@ -313,8 +333,9 @@ class SpecDecoder:
                     break
         torch.cuda.synchronize(self.device)
         total = time.perf_counter() - tic
-        self.base.check_fused_error()
-        self.draft.check_fused_error()
+        for m in (self.base, self.draft):
+            if m is not None:
+                m.check_fused_error()
         return self._result(first, i, total, max_tokens, clip, int(prompt.numel()))
 
     def _result(self, first: int, steps_run: int, total: float, max_tokens: int, clip: bool, prompt_len: int):
@@ -351,7 +372,8 @@ class SpecDecoder:
     def sync_offsets(self):
         c = self.read_ctl()
         self.base_cache.offset = c[CTL_BASE_LEN]
-        self.draft_cache.offset = c[CTL_DRAFT_LEN]
+        if self.draft_cache is not None:
+            self.draft_cache.offset = c[CTL_DRAFT_LEN]
         return c
 
 
@@ -545,12 +567,8 @@ def evaluate_posterior_greedy(logits: torch.Tensor, candidates: torch.Tensor):
 
 
 def accept_candidate(cache: KVCache, accept_indices: torch.Tensor, accept_length: int, offset: int):
-    """``mlx_eagle.py:349-376`` on the single-allocation cache."""
-    if accept_length > 0:
-        src = (offset + accept_indices.reshape(-1).to(torch.int64)).to(cache.data.device)
-        rows = cache.data[:, :, :, src].clone()
-        cache.data[:, :, :, offset + 1: offset + accept_length + 1] = rows
-    cache.offset = offset + accept_length + 1
+    """``mlx_eagle.py:349-376``: keep the root and the accepted rows of the last tree pass."""
+    cache.accept(accept_indices, accept_length, offset)
 
 
 def spec_step(dec: SpecDecoder):
@@ -565,7 +583,7 @@ def spec_step(dec: SpecDecoder):
             dec.ctl[CTL_BASE_LEN], dec.ctl[CTL_DRAFT_OFF])
 
 
-def generate_step(prompt: torch.Tensor, base_model: Model, draft_model: Model, prefill_step_size: int = 512,
+def generate_step(prompt: torch.Tensor, base_model: Model, draft_model: Optional[Model], prefill_step_size: int = 512,
                   k: int = 8, depth: int = 5, verify_num_tokens: int = 31, max_tokens: int = 128, tokenizer=None,
                   N: int = 20, use_graph: bool = True, verbose: bool = True, eos_token_id: Optional[int] = None,
                   clip: bool = False, temperature: float = 0.0, seed: int = 0):
@@ -573,6 +591,7 @@ def generate_step(prompt: torch.Tensor, base_model: Model, draft_model: Model, p
     (``verify_num_tokens`` is limited to 31 here) plus the two stop rules of ``SpecDecoder.generate``
     (``eos_token_id``, ``clip``) and, with ``temperature > 0``, sampling acceptance from the random stream ``seed``.  Builds a ``SpecDecoder`` for the request, captures
     its step graph and calls ``SpecDecoder.generate``; prints the reference's three summary lines.
+    ``draft_model=None`` decodes without speculation, one token per step.
     Returns the result dict of ``generate`` plus the decoder under ``"decoder"``."""
     rows = prompt.numel() + max_tokens + 8 * (depth + 2) + verify_num_tokens + 128
     rows = ((rows + 63) // 64) * 64
@@ -596,7 +615,7 @@ def parse_args(argv=None):
     """CLI flags of ``mlx_eagle.py:620-681``; a model is a local checkpoint directory or a shape preset
     (random-init weights: nothing can be downloaded where this was written)."""
     p = argparse.ArgumentParser(description="Tree speculative decoding on B200 with seeded random-init models.")
-    p.add_argument("--draft-model", type=str, default="qwen2-0.5b")
+    p.add_argument("--draft-model", type=str, default="qwen2-0.5b", help="'none': plain decoding, one token per step")
     p.add_argument("--base-model", type=str, default="qwen2-7b")
     p.add_argument("--prompt", type=str, required=True,
                    help="text (with a checkpoint that has a tokenizer), comma-separated token ids, or a number of seeded "
@@ -610,13 +629,15 @@ def parse_args(argv=None):
     p.add_argument("--clip", action="store_true", help="cut the output to exactly --max-tokens tokens")
     p.add_argument("--temp", type=float, default=0.0,
                    help="0: greedy acceptance (the reference); > 0: sampling acceptance at this temperature, stream --seed")
+    p.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
+                   help="activations of layer-list (hybrid) models; the 4-bit models are fp16")
     return p.parse_args(argv)
 
 
 def main(argv=None):
     """``python -m`` entry with the reference's flags (``mlx_eagle.py:683-756``).  ``--draft-model`` / ``--base-model``
-    name either a local MLX-format 4-bit checkpoint directory (``load.load``, the counterpart of ``mlx_utils.load``)
-    or a shape preset with seeded random-init weights; ``--prompt`` is text (needs the checkpoint's tokenizer),
+    name either a local checkpoint directory (``load.load``, the counterpart of ``mlx_utils.load``: MLX-format 4-bit, or a
+    layer-list design's) or a shape preset with seeded random-init weights; ``--prompt`` is text (needs the checkpoint's tokenizer),
     comma-separated token ids, or a count of seeded random tokens."""
     import os
     from . import load as _load
@@ -625,16 +646,16 @@ def main(argv=None):
 
     def get(name, seed):
         if os.path.isdir(name):
-            m, tok = _load.load(name, dev)
+            m, tok = _load.load(name, dev, dtype=args.dtype)
             return m.relayout(), tok
-        return Model.random_init(shape_preset(name), seed, dev).relayout(), None
+        return _load.random_model(name, seed, dev, dtype=args.dtype).relayout(), None
 
-    draft, _ = get(args.draft_model, args.seed + 1)
+    draft = None if args.draft_model == "none" else get(args.draft_model, args.seed + 1)[0]
     base, tokenizer = get(args.base_model, args.seed + 2)
     if args.prompt.isdigit():
         g = torch.Generator().manual_seed(args.seed)
-        ids = torch.randint(0, min(draft.args.vocab_size, base.args.vocab_size), (int(args.prompt),), generator=g,
-                            dtype=torch.int32)
+        vocab = min(m.args.vocab_size for m in (draft, base) if m is not None)
+        ids = torch.randint(0, vocab, (int(args.prompt),), generator=g, dtype=torch.int32)
     elif all(t.strip().lstrip("-").isdigit() for t in args.prompt.split(",")):
         ids = torch.tensor([int(t) for t in args.prompt.split(",")], dtype=torch.int32)
     elif tokenizer is not None:

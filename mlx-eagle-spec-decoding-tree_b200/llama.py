@@ -244,6 +244,18 @@ class KVCache:
             dtype=torch.float16, device=device)
         self.offset = 0
 
+    def reset(self):
+        """Forget the sequence (rows past ``offset`` are never read)."""
+        self.offset = 0
+
+    def accept(self, indices: torch.Tensor, accept_length: int, offset: int):
+        """Keep the root row and the accepted tree rows ``indices`` (``mlx_eagle.py:349-376``)."""
+        if accept_length > 0:
+            src = (offset + indices.reshape(-1).to(torch.int64)).to(self.data.device)
+            rows = self.data[:, :, :, src].clone()
+            self.data[:, :, :, offset + 1: offset + accept_length + 1] = rows
+        self.offset = offset + accept_length + 1
+
     def layer(self, i):
         return self.data[i, 0], self.data[i, 1]
 
@@ -265,6 +277,8 @@ class BatchKVCache:
 
 
 class Model:
+    stateful = False                                     # the cache is K/V rows only: rewinding its length undoes a pass
+
     def __init__(self, args: ModelArgs, layers: List[dict], embed: QLinear, norm: torch.Tensor,
                  lm_head: Optional[QLinear], device):
         self.args = args
@@ -663,6 +677,21 @@ class Model:
         vl = self.vocab_local                      # a tensor-parallel shard produces its slice of the vocabulary
         return self.logits[:rows] if vl == a.vocab_size else self.logits.view(-1)[: rows * vl].view(rows, vl)
 
+    # ------------------------------------------------------------------ hooks of the decoding loop
+    def commit_catchup(self, cache: KVCache, accept: torch.Tensor):
+        """After a draft's catch-up pass (nothing to do: rows are in the cache, the loop moves the length)."""
+
+    def commit_accepted(self, cache: KVCache, accept_rows: torch.Tensor, ctl: torch.Tensor, tree_rows: int):
+        """After acceptance: move the accepted nodes' K/V rows together."""
+        a, p = self.args, _lib.ptr
+        _lib.check(_lib.lib().b200_kv_compact(p(cache.data), a.num_hidden_layers, a.num_key_value_heads, cache.rows, a.head_dim,
+                                              p(accept_rows), p(ctl), _lib.stream_ptr(self.device)), "b200_kv_compact")
+
+    def argmax_rows(self, logits: torch.Tensor, rows: int, key: torch.Tensor):
+        """Greedy token of every row of a pass's logits, as ordering keys."""
+        _lib.check(_lib.lib().b200_logits_argmax(_lib.ptr(logits), rows, self.vocab_local, _lib.ptr(key),
+                                                 _lib.stream_ptr(self.device)), "b200_logits_argmax")
+
     # ------------------------------------------------------------------ prompt ingestion, 128 rows per weight read
     def can_prefill_large_m(self) -> bool:
         """True when a causal prompt can go through ``b200_qmm_umma`` 128 rows at a time: weights in the
@@ -772,14 +801,18 @@ class Model:
     # ------------------------------------------------------------------ reference-style call
     def __call__(self, inputs: torch.Tensor, cache: Optional[KVCache] = None, mask: Optional[torch.Tensor] = None,
                  position_ids: Optional[Union[torch.Tensor, int]] = None, flat_rope: bool = False,
-                 logits_last_only: bool = False) -> torch.Tensor:
+                 logits_last_only: bool = False, want=None) -> torch.Tensor:
         """``logits (1, L, V)``; the argument meanings follow ``mlx_llama.py:298-313`` / ``:121-196``.
 
         ``mask`` is the additive matrix ``(1,1,L,cache.offset+L)`` of 0 / -inf the reference passes
         (``mlx_eagle.py:177,338``); ``None`` means causal.  Calls longer than 32 tokens (prompt
         ingestion) are split into passes of 32, which is only possible with the causal mask.
-        ``logits_last_only`` (an addition) returns only the last token's logits ``(1, 1, V)``.
+        ``logits_last_only`` (an addition) returns only the last token's logits ``(1, 1, V)``, ``want`` (another) those of the
+        given places among the tokens (None when empty).
         """
+        if want is not None:
+            full = self(inputs, cache, mask, position_ids, flat_rope, logits_last_only=not len(want))
+            return full[:, list(want)] if len(want) else None
         if cache is None:
             raise _lib.B200Error("a KVCache is required (the reference's cache-less branch is not on this path)")
         inputs = inputs.reshape(-1).to(torch.int32)

@@ -1,4 +1,7 @@
-"""Checkpoint ingestion: MLX-format 4-bit checkpoints -> ``llama.Model``.
+"""Checkpoint ingestion: MLX-format 4-bit checkpoints -> ``llama.Model``, layer-list checkpoints -> ``hybrid.HybridModel``.
+
+``load_model`` picks the model class from ``config.json``: ``architecture`` (``ARCHITECTURES``) or, for the Hugging Face
+style configurations, ``model_type`` (``MODEL_TYPES``).
 
 The counterpart of the reference's ``mlx_utils.py:59-181`` (``load_model`` / ``load``): a directory with
 ``config.json`` (Hugging Face keys plus ``"quantization": {"group_size": 64, "bits": 4}``) and
@@ -32,7 +35,8 @@ import numpy as np
 import torch
 
 from . import _lib
-from .llama import Model, ModelArgs, QLinear
+from .hybrid import HybridArgs, HybridModel, preset_config
+from .llama import Model, ModelArgs, QLinear, shape_preset
 
 _DTYPES = {"U32": (np.uint32, 4), "I32": (np.int32, 4), "F16": (np.float16, 2), "F32": (np.float32, 4),
            "BF16": (np.uint16, 2), "U8": (np.uint8, 1), "I64": (np.int64, 8)}
@@ -108,18 +112,12 @@ def _f16(t: torch.Tensor) -> torch.Tensor:
     return t.to(torch.float16).contiguous()
 
 
-def load_model(model_path: str, device, model_config: Optional[dict] = None) -> Model:
-    """``mlx_utils.load_model`` (``:59-141``) for this library: reads ``config.json`` and every weight file of
-    the directory and returns a ``Model`` on ``device`` (row-major packed weights; call ``relayout()`` for the
-    persistent-kernel path)."""
+def read_config(model_path: str) -> dict:
     with open(os.path.join(model_path, "config.json")) as f:
-        config = json.load(f)
-    config.update(model_config or {})
-    q = config.get("quantization")
-    if not q or int(q.get("bits", 0)) != 4 or int(q.get("group_size", 0)) != 64:
-        raise _lib.B200Error("only 4-bit / group-64 quantised checkpoints are supported (config.json: quantization)")
-    if config.get("model_type") not in ("llama", "qwen2"):
-        raise _lib.B200Error(f"no implementation for model architecture {config.get('model_type')!r}")
+        return json.load(f)
+
+
+def _read_weights(model_path: str) -> Dict[str, torch.Tensor]:
     files = sorted(glob.glob(os.path.join(model_path, "model*.safetensors"))) or \
         sorted(glob.glob(os.path.join(model_path, "weight*.safetensors")))
     if not files:
@@ -127,7 +125,46 @@ def load_model(model_path: str, device, model_config: Optional[dict] = None) -> 
     w: Dict[str, torch.Tensor] = {}
     for wf in files:
         w.update(read_safetensors(wf))
-    w = {k: v for k, v in w.items() if "rotary_emb.inv_freq" not in k}            # Model.sanitize of the reference
+    return w
+
+
+def model_builder(config: dict):
+    """(builder, name of its kernel library, runs in fp32) of a configuration; raises for an unknown architecture."""
+    if "architecture" in config:
+        if config["architecture"] in ARCHITECTURES:
+            return ARCHITECTURES[config["architecture"]]
+        raise _lib.B200Error(f"no implementation for model architecture {config['architecture']!r}")
+    if config.get("model_type") in MODEL_TYPES:
+        return MODEL_TYPES[config["model_type"]]
+    raise _lib.B200Error(f"no implementation for model architecture {config.get('model_type')!r}")
+
+
+def load_model(model_path: str, device, model_config: Optional[dict] = None, dtype: str = "bfloat16"):
+    """``mlx_utils.load_model`` (``:59-141``) for this library: reads ``config.json`` and every weight file of
+    the directory and returns the model on ``device``.  4-bit models: row-major packed weights, call ``relayout()`` for the
+    persistent-kernel path.  ``dtype`` is the activation type of models that have a choice."""
+    config = read_config(model_path)
+    config.update(model_config or {})
+    return model_builder(config)[0](model_path, config, device, dtype)
+
+
+def _load_hybrid(model_path: str, config: dict, device, dtype: str) -> HybridModel:
+    return HybridModel(HybridArgs.from_config(config), _read_weights(model_path), device, dtype)
+
+
+def random_model(name: str, seed: int, device, dtype: str = "bfloat16"):
+    """A model of a named shape with seeded random weights (``llama.shape_preset`` or ``hybrid.preset_config``)."""
+    try:
+        return Model.random_init(shape_preset(name), seed, device)
+    except KeyError:
+        return HybridModel.random_init(HybridArgs.from_config(preset_config(name)), seed, device, dtype=dtype)
+
+
+def _load_quantised(model_path: str, config: dict, device, dtype: str) -> Model:
+    q = config.get("quantization")
+    if not q or int(q.get("bits", 0)) != 4 or int(q.get("group_size", 0)) != 64:
+        raise _lib.B200Error("only 4-bit / group-64 quantised checkpoints are supported (config.json: quantization)")
+    w = {k: v for k, v in _read_weights(model_path).items() if "rotary_emb.inv_freq" not in k}            # Model.sanitize of the reference
     args = _args_from_config(config)
     dev = torch.device(device)
     H, I, hd = args.hidden_size, args.intermediate_size, args.head_dim
@@ -172,12 +209,17 @@ def load_model(model_path: str, device, model_config: Optional[dict] = None) -> 
     return Model(args, layers, embed, _f16(w["model.norm.weight"]).to(dev), lm_head, dev)
 
 
-def load(path: str, device, tokenizer_config: Optional[dict] = None, model_config: Optional[dict] = None):
+# name in config.json -> (builder, kernel library, does it run in fp32)
+MODEL_TYPES = {"llama": (_load_quantised, "eagle", False), "qwen2": (_load_quantised, "eagle", False)}
+ARCHITECTURES = {"Zaverax": (_load_hybrid, "hybrid", True)}
+
+
+def load(path: str, device, tokenizer_config: Optional[dict] = None, model_config: Optional[dict] = None, dtype: str = "bfloat16"):
     """``mlx_utils.load`` (``:144-181``): ``(model, tokenizer)``.  ``path`` must be a local directory (nothing is
     downloaded).  The tokenizer comes from ``transformers`` when the directory holds tokenizer files, else None."""
     if not os.path.isdir(path):
         raise FileNotFoundError(f"{path}: not a local checkpoint directory (downloads are not supported here)")
-    model = load_model(path, device, model_config)
+    model = load_model(path, device, model_config, dtype)
     tokenizer = None
     if any(os.path.exists(os.path.join(path, n)) for n in ("tokenizer.json", "tokenizer.model", "tokenizer_config.json")):
         from transformers import AutoTokenizer
