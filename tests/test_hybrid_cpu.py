@@ -1,0 +1,172 @@
+"""Layer-list decoders, what needs no GPU: configuration, tables, ABI, oracle sanity, runner conventions."""
+import ctypes
+import json
+import os
+import re
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+import torch
+
+import hybrid_cases as hc
+from oracle import hybrid_ref
+
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+
+
+def test_header_symbols_are_exported(be):
+    text = re.sub(r"/\*.*?\*/", "", open(os.path.join(ROOT, "include", "b200_hybrid.h")).read(), flags=re.S)
+    names = set(re.findall(r"\b(b200_hybrid_[a-z0-9_]+)\s*\(", text))
+    assert {"b200_hybrid_forward", "b200_hybrid_commit", "b200_hybrid_linear"} <= names
+    for n in names:
+        assert hasattr(be._lib.hybrid(), n), n
+
+
+def test_struct_mirrors(be):
+    L = be._lib
+    assert ctypes.sizeof(L.Linear) == 24
+    assert ctypes.sizeof(L.HybridLayer) == 10 * 4 + 3 * 4 + 4 * 4 + 4 + 6 * 8 + 4 * 24
+    assert ctypes.sizeof(L.HybridRun) == 8 + 7 * 8
+    assert ctypes.sizeof(L.HybridPass) == 8 * 4 + 11 * 8
+
+
+def test_bad_arguments_are_refused_before_any_launch(be):
+    L = be._lib.hybrid()
+    m, p = be._lib.HybridModelDesc(), be._lib.HybridPass()
+    assert L.b200_hybrid_forward(ctypes.byref(m), ctypes.byref(p), None) == -1
+    assert L.b200_hybrid_commit(ctypes.byref(m), None, 0, None, None, 0, None, 0, None) == -1
+
+
+def test_runs_of_a_loop(be):
+    c = hc.mixed()
+    a = be.HybridArgs.from_config(c)
+    assert a.runs == [(0, False), (1, False), (2, False), (3, True), (1, False), (2, False), (3, False), (4, False)]
+    assert [i for i, _ in hybrid_ref.layer_order(c)] == [i for i, _ in a.runs]
+    one = hc.mixed()
+    one["loop"] = dict(start=0, stop=5, times=3)
+    a = be.HybridArgs.from_config(one)
+    assert [i for i, _ in a.runs] == [0, 1, 2, 3, 4] * 3 and [j for j, (_, s) in enumerate(a.runs) if s] == [4, 9]
+    one["loop"] = None
+    assert be.HybridArgs.from_config(one).num_hidden_layers == 5
+
+
+def test_unknown_parts_raise(be):
+    c = hc.mixed()
+    c["layers"][0]["type"] = "other"
+    with pytest.raises(be._lib.B200Error):
+        be.HybridArgs.from_config(c)
+    with pytest.raises(be._lib.B200Error):
+        be.load.model_builder({"architecture": "other"})
+    with pytest.raises(be._lib.B200Error):
+        be.load.model_builder({"model_type": "other"})
+
+
+def test_checkpoint_tensors_are_checked(be):
+    c = hc.mixed()
+    w = hc.weights(c)
+    assert set(w) == set(be.hybrid.weight_shapes(be.HybridArgs.from_config(c)))
+    bad = dict(w)
+    bad.pop("l1.mix.g")
+    with pytest.raises(be._lib.B200Error):
+        be.HybridModel(be.HybridArgs.from_config(c), bad, "cpu")
+    bad = dict(w, **{"l1.mix.g": w["l1.mix.g"][1:]})
+    with pytest.raises(be._lib.B200Error):
+        be.HybridModel(be.HybridArgs.from_config(c), bad, "cpu")
+
+
+def test_cache_parts_do_not_overlap(be):
+    c = hc.mixed()
+    m = be.HybridModel(be.HybridArgs.from_config(c), hc.weights(c), "cpu")
+    rows = 77
+    lay = m.cache_layout(rows)
+    parts = []
+    for r, (li, _) in zip(lay.runs, m.args.runs):
+        mx = c["layers"][li]["mixer"]
+        parts.append((r.conv_off, 4 * 2 * c["width"]))
+        if c["layers"][li]["type"] == "hgrn2":
+            parts.append((r.state_off, 4 * mx["heads"] * mx["dim"] * mx["vdim"]))
+        else:
+            parts.append((r.k_off, 2 * mx["kv_heads"] * rows * 2 * -(-mx["dim"] // 16) * 16))
+            parts.append((r.v_off, 2 * mx["kv_heads"] * rows * -(-mx["vdim"] // 16) * 16))
+    parts.sort()
+    for (a, n), (b, _) in zip(parts, parts[1:] + [(lay.nbytes, 0)]):
+        assert a % 256 == 0 and a + n <= b
+    states = [r.state_off for r, (li, _) in zip(lay.runs, m.args.runs) if c["layers"][li]["type"] == "hgrn2"]
+    assert len(set(states)) == len(states) and max(states) < lay.state_bytes <= min(
+        r.k_off for r, (li, _) in zip(lay.runs, m.args.runs) if c["layers"][li]["type"] == "attention")
+    cache = m.make_cache(rows)
+    cache.data.fill_(1)
+    cache.offset = 5
+    cache.reset()
+    assert cache.offset == 0 and int(cache.data[: lay.state_bytes].sum()) == 0 and int(cache.data[lay.state_bytes]) == 1
+
+
+def test_differential_constants(be):
+    c = hc.config([hc.attention(diff=0.35)])
+    w = hc.weights(c, 3)
+    m = be.HybridModel(be.HybridArgs.from_config(c), w, "cpu")
+    n = hc.as_numpy(w)
+    lam = hybrid_ref.differential_lambda(*(n["l0.mix." + k] for k in ("lq1", "lk1", "lq2", "lk2")), 0.35)
+    assert abs(m.layers[0].lambda_ - lam) < 1e-6 and abs(m.layers[0].out_scale - 0.65) < 1e-6
+    assert m.layers[0].window == 20 and m.layers[0].keep_first == 2
+
+
+def test_oracle_mechanisms():
+    """The restatement against closed forms."""
+    rng = np.random.default_rng(0)
+    h = rng.standard_normal((6, 4))
+    w = np.zeros((4, 3))
+    w[:, 1] = 2.0                                            # the middle of three taps: the previous token
+    out = hybrid_ref.causal_conv_residual(h, w)
+    assert np.allclose(out[0], h[0]) and np.allclose(out[1:], h[1:] + 2 * h[:-1])
+    f, q, v = rng.uniform(0.1, 0.9, (5, 3)), rng.standard_normal((5, 3)), rng.standard_normal((5, 2))
+    o = hybrid_ref.gated_recurrence(q, f, v)
+    want = sum(np.sum(q[4] * (1 - f[j]) * np.prod(f[j + 1:5], axis=0)) * v[j] for j in range(5))
+    assert np.allclose(o[4], want)
+    vis = [[hybrid_ref.visible(i, j, 3, 2) for j in range(8)] for i in range(8)]
+    assert [j for j in range(8) if vis[7][j]] == [0, 1, 5, 6, 7] and [j for j in range(8) if vis[1][j]] == [0, 1]
+    z = rng.standard_normal((2, 9))
+    y = hybrid_ref.polynorm(z, (0.0, 0.0, 1.0, 0.5), 0.0)
+    assert np.allclose(np.mean((y - 0.5) ** 2, axis=1), 1.0)
+
+
+def test_replay_keeps_and_reuses_caches(be):
+    class Fake:
+        made = 0
+
+        def make_cache(self, rows):
+            Fake.made += 1
+
+            class C:
+                def reset(self):
+                    self.seen = []
+            return C()
+
+        def __call__(self, toks, cache, want):
+            cache.seen += toks.tolist()
+            return torch.tensor([[[float(sum(cache.seen))]] * len(want)]).reshape(1, len(want), 1) if want else None
+
+        def check_fused_error(self):
+            pass
+
+    r = be.trace.Replay(Fake(), 64)
+    assert r.step(dict(entries=[dict(id="a", tokens=[1, 2], want=[])], end=[])) is None
+    assert r.step(dict(entries=[dict(id="b", tokens=[5], want=[0]), dict(id="a", tokens=[3], want=[0])], end=["a"])).flatten().tolist() == [5.0, 6.0]
+    assert r.step(dict(entries=[dict(id="c", tokens=[7], want=[0])], end=["c", "b"])).flatten().tolist() == [7.0]
+    assert Fake.made == 2 and len(r.free) == 2 and not r.live
+
+
+def test_runner_refuses_fp32_where_there_is_none(tmp_path):
+    (tmp_path / "config.json").write_text(json.dumps({"model_type": "llama"}))
+    p = subprocess.run([sys.executable, os.path.join(ROOT, "bin", "trace_run"), "--model", str(tmp_path), "--dtype", "float32", "--out",
+                        str(tmp_path)], input="", capture_output=True, text=True, timeout=300)
+    assert p.returncode == 3
+
+
+def test_presets(be):
+    for n in ("tiny-zaverax", "zaverax-1b", "zaverax-8b"):
+        be.HybridArgs.from_config(be.hybrid.preset_config(n))
+    with pytest.raises(KeyError):
+        be.hybrid.preset_config("none")
