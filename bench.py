@@ -1,6 +1,6 @@
 """Benchmark of the tree speculative decoding hot path.
 
-    python bench.py [--gpus N] [--steps K] [--warmup W] [--impl b200|reference] [--workload c3|c2|c4|tp70b|tp7b]
+    python bench.py [--gpus N] [--steps K] [--warmup W] [--impl b200|reference] [--workload c3|c2|c4|tp70b|tp7b|hybrid]
 
 Default workload ``c3`` (N = 1 and every rank at N > 1): full speculative decode steps, greedy, Qwen2-7B-shape
 4-bit target + Qwen2-0.5B-shape 4-bit draft (random-init weights, seeded), 256-token seeded random prompt,
@@ -727,6 +727,117 @@ def batched_requests_numbers(torch, be, base, draft, depth, verify, prompt_len, 
     return out
 
 
+# layer-list design beside the 4-bit model of the same width, feed-forward and layer count
+HYBRID_PAIRS = {"1b": ("zaverax-1b", "llama3.2-1b"), "8b": ("zaverax-8b", "llama3-8b")}
+
+
+def hybrid_numbers(torch, be, name, dev, prompt_len, steps, layers=0):
+    """Plain decoding (one token per step, CUDA graph) and prompt ingestion of one model with random weights, and how far
+    each is from its roofline: the bytes a step must stream over the HBM peak, the prompt's multiply-adds over the
+    tensor-core peak."""
+    import dataclasses
+    peak, _ = _peaks()
+    mpath = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    tensor_peak = 1590.0
+    if os.path.exists(mpath):
+        with open(mpath) as f:
+            tensor_peak = float(json.load(f).get("bf16_tflops", tensor_peak))
+    if name.startswith("zaverax"):
+        args = be.HybridArgs.from_config(be.hybrid.preset_config(name))
+        if layers:
+            args = dataclasses.replace(args, layers=args.layers[:layers])
+        m = be.HybridModel.random_init(args, 7, dev, max_rows=max(256, prompt_len))
+        state = m.cache_layout(64).state_bytes
+        kv = 0
+        for li, _ in args.runs:
+            sp = args.layers[li]
+            if sp.type == "attention":
+                mx = sp.mixer
+                keys = min(prompt_len, mx["mask"]["size"])
+                kv += 2 * keys * mx["kv_heads"] * (2 * mx["dim"] + mx["vdim"])
+        stream = m.linear_weight_bytes() + kv + 2 * state              # the states are read and written
+        macs = m.linear_weight_bytes() // 2
+        head = args.vocab_size * args.width
+    else:
+        shape = be.shape_preset(name)
+        if layers:
+            shape = dataclasses.replace(shape, num_hidden_layers=layers)
+        m = be.Model.random_init(shape, 7, dev).relayout()
+        m.prefill_graphs = False                        # prompt chunks launched one by one (GPU-bound at these sizes)
+        stream = m.linear_weight_bytes() + 4 * shape.num_hidden_layers * prompt_len * shape.num_key_value_heads * shape.head_dim
+        macs = int(m.linear_weight_bytes() / 0.5625)
+        head = shape.vocab_size * shape.hidden_size
+    dec = be.SpecDecoder(m, None, 0, 0, ((prompt_len + steps + 192 + 63) // 64) * 64)
+    g = torch.Generator().manual_seed(3)
+    prompt = torch.randint(0, m.args.vocab_size, (prompt_len,), generator=g, dtype=torch.int32)
+    dec.warmup()
+
+    def timed(fn, reps):
+        fn()
+        fn()
+        torch.cuda.synchronize()
+        ts = []
+        for _ in range(reps):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1) / 1e3)
+        return statistics.median(ts)
+
+    def ingest():
+        dec.base_cache.reset()
+        m(prompt, dec.base_cache, logits_last_only=True)
+
+    t_prompt = timed(ingest, 9)
+    dec.prefill(prompt)
+    ctl0, y0 = dec.ctl.clone(), dec.y.clone()
+
+    def decode():
+        dec.ctl.copy_(ctl0)
+        dec.y.copy_(y0)
+        for _ in range(steps):
+            dec.replay()
+
+    t_step = timed(decode, 5) / steps
+    m.check_fused_error()
+    out = {"model": name, "layers": m.args.num_hidden_layers, "weights": "bf16" if name.startswith("zaverax") else "4 bit",
+           "decode_tokens_per_s": round(1 / t_step, 1), "decode_ms": round(t_step * 1e3, 4), "decode_bytes": stream,
+           "decode_frac_of_hbm": round(stream / t_step / 1e9 / peak, 3), "prompt_tokens": prompt_len,
+           "prompt_tokens_per_s": round(prompt_len / t_prompt), "prompt_ms": round(t_prompt * 1e3, 3),
+           "prompt_frac_of_tensor": round(2 * ((macs - head) * prompt_len + head) / t_prompt / 1e12 / tensor_peak, 3)}
+    del dec, m
+    torch.cuda.empty_cache()
+    return out
+
+
+def run_hybrid(args, torch, be, dev, local_rank):
+    """``--workload hybrid``: the layer-list design at two sizes beside the 4-bit model of equal size (plain decoding
+    at the prompt's context length, prompt ingestion); one JSON line, ``value`` = decoded tokens/s of the 8b-size design."""
+    steps = args.steps
+    if args.hybrid_model:
+        print(json.dumps(hybrid_numbers(torch, be, args.hybrid_model, dev, 1024, steps, args.layers)))
+        return
+    sampler = ClockSampler(local_rank)
+    sampler.start()
+    res = {}
+    for k, pair in HYBRID_PAIRS.items():
+        res[k] = []
+        for n in pair:                                  # a process of its own each: nothing of one model is left for the next
+            r = subprocess.run([sys.executable, os.path.abspath(__file__), "--workload", "hybrid", "--hybrid-model", n, "--steps", str(steps),
+                                "--layers", str(args.layers)], capture_output=True, text=True, timeout=900)
+            if r.returncode != 0:
+                raise SystemExit(f"{n}: {r.stderr[-2000:]}")
+            res[k].append(json.loads(r.stdout.strip().splitlines()[-1]))
+    clocks = sampler.stop()
+    print(json.dumps({"metric": "plain decoding tokens/s (layer-list design, 8B-size layers, bf16, random weights)",
+                      "value": res["8b"][0]["decode_tokens_per_s"], "unit": UNIT, "n_gpus": 1, "steps": steps,
+                      "ms_per_step": res["8b"][0]["decode_ms"], "higher_is_better": True, "dtype": "bf16", "data": "synthetic",
+                      "config": {"model": "zaverax-8b", "prompt": 1024, "peaks": _peaks()[1],
+                                 "l2": "weights of one step exceed L2"}, "clocks": clocks, "pairs": res}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -741,7 +852,8 @@ def main():
                     help="only one model's forward kernel (small profiling case with --layers): the target at 16 rows, or "
                          "with --draft the draft at 8 rows")
     ap.add_argument("--draft", action="store_true", help="with --roofline-only: the draft model's pass instead of the target's")
-    ap.add_argument("--layers", type=int, default=0, help="with --roofline-only: number of decoder layers (0 = all)")
+    ap.add_argument("--layers", type=int, default=0, help="with --roofline-only or --workload hybrid: number of decoder layers (0 = all)")
+    ap.add_argument("--hybrid-model", default="", help="with --workload hybrid: only this preset")
     ap.add_argument("--operator-sweep", action="store_true",
                     help="only time the two matmul operators (mma.sync streaming kernel, tcgen05 kernel) at big layer shapes")
     ap.add_argument("--qmm-sweep", action="store_true", help="only the 8192 x 2048 operator sweep at 1..32 rows")
@@ -749,9 +861,10 @@ def main():
     ap.add_argument("--launches", type=int, default=100, help="with --qmm-sweep: timed launches per kernel and row count")
     ap.add_argument("--min-seconds", type=float, default=MIN_TIMED_SECONDS,
                     help="repeat the block of --steps steps until this much time has been measured (0: three blocks; profiling)")
-    ap.add_argument("--workload", default="c3", choices=["streams"] + sorted(STREAM_WORKLOADS) + sorted(TP_WORKLOADS),
+    ap.add_argument("--workload", default="c3", choices=["streams", "hybrid"] + sorted(STREAM_WORKLOADS) + sorted(TP_WORKLOADS),
                     help="c3 (= streams, the default): one independent request stream per GPU; c2: draft-only tree build; c4: "
-                         "Llama-3-8B/3.2-1B shapes, prompt 1024; tp70b / tp7b: one stream with the target cut across all ranks")
+                         "Llama-3-8B/3.2-1B shapes, prompt 1024; tp70b / tp7b: one stream with the target cut across all ranks; hybrid: "
+                         "the layer-list design beside the 4-bit models of equal size (one GPU)")
     args = ap.parse_args()
     if args.workload == "streams":
         args.workload = "c3"
@@ -773,6 +886,9 @@ def main():
         return
     torch.cuda.set_device(local_rank)
     dev = torch.device("cuda", local_rank)
+    if args.workload == "hybrid":
+        run_hybrid(args, torch, be, dev, local_rank)
+        return
     if args.operator_sweep:
         print(json.dumps({"operator_sweep": operator_sweep(torch, be, dev, reps=max(1, min(args.steps, 20)))}))
         return

@@ -51,22 +51,26 @@ struct KeyWalk {
         nc = ns + prefix - wstart;
         total = nc + (p.tree ? p.tail : 0);
     }
+    __device__ __forceinline__ int blocks() const { return (total + kKeys - 1) / kKeys; }
+    __device__ __forceinline__ int per_split(const AttnParams& p) const { return (blocks() + p.splits - 1) / p.splits; }
     __device__ __forceinline__ int row(int u) const { return u < ns ? u : (u < nc ? wstart + u - ns : prefix + u - nc); }
 };
 
-template <typename T, int QN, int CR>
+template <typename T, int QN, int CR>    // query vectors (at most), columns per thread
 __global__ void __launch_bounds__(kRowThreads) attention_rows_kernel(const AttnParams p) {
-    pdl_wait();
     pdl_launch_dependents();
+    pdl_wait();
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    const int KE = p.maps * p.dp, KP = KE + 16 / (int)sizeof(T);         // padded key row
+    constexpr int VE = 16 / (int)sizeof(T), SP = kKeys + 4;              // elements of 16 bytes, pitch of a score row
+    const int KE = p.maps * p.dp, KP = KE + VE;                          // padded key row
     float* sq = reinterpret_cast<float*>(smem_raw);                      // [QN][dp]
-    float* sc = sq + QN * p.dp;                                          // [QN][kKeys]
-    float* sm = sc + QN * kKeys;                                         // [QN] running max
+    float* sc = sq + QN * p.dp;                                          // [QN][SP]
+    float* sm = sc + QN * SP;                                            // [QN] running max
     float* sl = sm + QN;                                                 // [QN] running sum
-    float* sr = sl + QN;                                                 // [QN] rescale factor of this block
+    float* sr = sl + QN;                                                 // [2 QN] rescale factor of this block
     int* srow = reinterpret_cast<int*>(sr + 2 * QN);                     // [kKeys] cache row of the block's keys, -1: not visible
     T* sk = reinterpret_cast<T*>(srow + kKeys);                          // [kKeys][KP]
+    T* sv = sk + kKeys * KP;                                             // [kKeys][vp]
     const int split = blockIdx.x, g = blockIdx.y / p.qgroups, qg = blockIdx.y % p.qgroups, m = blockIdx.z;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int R = p.H / p.G;
@@ -74,11 +78,11 @@ __global__ void __launch_bounds__(kRowThreads) attention_rows_kernel(const AttnP
     const int nh = min(p.hpg, R - qg * p.hpg), nq = nh * p.maps;
     KeyWalk kw;
     kw.init(p, m);
-    const int nb = (kw.total + kKeys - 1) / kKeys, per = (nb + p.splits - 1) / p.splits;
-    const int b0 = split * per, b1 = min(nb, b0 + per);
+    const int nb = kw.blocks(), per = kw.per_split(p), b0 = split * per, b1 = min(nb, b0 + per);
+    if (b0 >= b1) return;                                                // the merge knows which splits hold something
 
     const T* qrow = static_cast<const T*>(p.q) + (size_t)m * p.q_pitch + (size_t)h0 * p.maps * p.dp;
-    for (int i = tid; i < QN * p.dp; i += kRowThreads) sq[i] = (i < nq * p.dp && i % p.dp < p.dim) ? to_f32<T>(qrow[i]) * p.scale_log2 : 0.f;
+    for (int i = tid; i < QN * p.dp; i += kRowThreads) sq[i] = i < nq * p.dp ? to_f32<T>(qrow[i]) * p.scale_log2 : 0.f;
     for (int i = tid; i < QN; i += kRowThreads) { sm[i] = -INFINITY; sl[i] = 0.f; }
     float acc[QN][CR];
 #pragma unroll
@@ -91,11 +95,10 @@ __global__ void __launch_bounds__(kRowThreads) attention_rows_kernel(const AttnP
 
     for (int b = b0; b < b1; b++) {
         __syncthreads();
-        const int u0 = b * kKeys, cnt = min(kKeys, kw.total - u0);
         if (tid < kKeys) {
+            const int u = b * kKeys + tid;
             int r = -1;
-            if (tid < cnt) {
-                const int u = u0 + tid;
+            if (u < kw.total) {
                 r = kw.row(u);
                 if (u >= kw.nc) {
                     const int j = u - kw.nc, tp = p.tail_pos[j];
@@ -106,39 +109,49 @@ __global__ void __launch_bounds__(kRowThreads) attention_rows_kernel(const AttnP
             srow[tid] = r;
         }
         __syncthreads();
-        constexpr int VE = 16 / (int)sizeof(T);
-        const int vpr = KE / VE;
-        for (int i = tid; i < kKeys * vpr; i += kRowThreads) {
-            const int k = i / vpr, c = i - k * vpr, r = srow[k];
-            uint4 v = make_uint4(0, 0, 0, 0);
-            if (r >= 0) v = *reinterpret_cast<const uint4*>(kbase + (size_t)r * KE + c * VE);
-            *reinterpret_cast<uint4*>(sk + k * KP + c * VE) = v;
+        for (int k = warp; k < kKeys; k += kRowThreads / 32) {           // a warp per key row, 16 bytes per lane
+            const int r = srow[k];
+            for (int c = lane; c * VE < KE + p.vp; c += 32) {
+                const bool key = c * VE < KE;
+                T* dst = key ? sk + k * KP + c * VE : sv + k * p.vp + (c * VE - KE);
+                const T* src = key ? kbase + (size_t)r * KE + c * VE : vbase + (size_t)r * p.vp + (c * VE - KE);
+                if (r >= 0) cp_async16(smem_u32(dst), src);
+                else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+            }
         }
+        asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;\n" ::: "memory");
         __syncthreads();
         {
             const int k = tid & (kKeys - 1);
             const bool vis = srow[k] >= 0;
             for (int qi = tid / kKeys; qi < nq; qi += kRowThreads / kKeys) {
-                const T* kr = sk + k * KP + (qi % p.maps) * p.dp;
+                const T* kr = sk + k * KP + (p.maps == 2 ? (qi & 1) * p.dp : 0);
                 const float* qv = sq + qi * p.dp;
-                float s = 0.f;
+                float s0 = 0.f, s1 = 0.f;
+#pragma unroll 4
                 for (int c = 0; c < p.dp; c += VE) {
                     const uint4 raw = *reinterpret_cast<const uint4*>(kr + c);
                     const T* kv = reinterpret_cast<const T*>(&raw);
 #pragma unroll
-                    for (int e = 0; e < VE; e++) s = fmaf(qv[c + e], to_f32<T>(kv[e]), s);
+                    for (int e = 0; e < VE; e += 4) {
+                        const float4 q4 = *reinterpret_cast<const float4*>(qv + c + e);
+                        s0 = fmaf(q4.x, to_f32<T>(kv[e]), s0);
+                        s1 = fmaf(q4.y, to_f32<T>(kv[e + 1]), s1);
+                        s0 = fmaf(q4.z, to_f32<T>(kv[e + 2]), s0);
+                        s1 = fmaf(q4.w, to_f32<T>(kv[e + 3]), s1);
+                    }
                 }
-                sc[qi * kKeys + k] = vis ? s : -INFINITY;
+                sc[qi * SP + k] = vis ? s0 + s1 : -INFINITY;
             }
         }
         __syncthreads();
         for (int qi = warp; qi < nq; qi += kRowThreads / 32) {
-            const float a0 = sc[qi * kKeys + lane], a1 = sc[qi * kKeys + lane + 32];
+            const float a0 = sc[qi * SP + lane], a1 = sc[qi * SP + lane + 32];
             const float mo = sm[qi], mn = fmaxf(mo, warp_max(fmaxf(a0, a1)));
             const float base = mn == -INFINITY ? 0.f : mn;
             const float p0 = exp2f(a0 - base), p1 = exp2f(a1 - base);
-            sc[qi * kKeys + lane] = p0;
-            sc[qi * kKeys + lane + 32] = p1;
+            sc[qi * SP + lane] = p0;
+            sc[qi * SP + lane + 32] = p1;
             const float ls = warp_sum(p0 + p1);
             __syncwarp();
             if (lane == 0) {
@@ -156,28 +169,26 @@ __global__ void __launch_bounds__(kRowThreads) attention_rows_kernel(const AttnP
 #pragma unroll
                 for (int i = 0; i < QN; i++)
                     if (i < nq) acc[i][c] *= sr[i];
-#pragma unroll 4
-                for (int k = 0; k < cnt; k++) {
-                    const int r = srow[k];
-                    if (r < 0) continue;
-                    const float v = to_f32<T>(vbase[(size_t)r * p.vp + col]);
+#pragma unroll 2
+                for (int k = 0; k < kKeys; k += 4) {                     // rows that are not visible: weight 0, value 0
+                    float v[4];
+#pragma unroll
+                    for (int e = 0; e < 4; e++) v[e] = to_f32<T>(sv[(k + e) * p.vp + col]);
 #pragma unroll
                     for (int i = 0; i < QN; i++)
-                        if (i < nq) acc[i][c] = fmaf(sc[i * kKeys + k], v, acc[i][c]);
+                        if (i < nq) {
+                            const float4 w = *reinterpret_cast<const float4*>(sc + i * SP + k);
+                            acc[i][c] = fmaf(w.x, v[0], fmaf(w.y, v[1], fmaf(w.z, v[2], fmaf(w.w, v[3], acc[i][c]))));
+                        }
                 }
             }
         }
-    }
-    __syncthreads();
-    for (int i = 0; i < QN; i++) {
-        if (i >= nq) break;
-        float* dst = p.part + (((size_t)m * p.H * p.maps + (size_t)h0 * p.maps + i) * p.splits + split) * (p.vp + 2);
-        if (tid == 0) { dst[0] = sm[i]; dst[1] = sl[i]; }
     }
 #pragma unroll
     for (int i = 0; i < QN; i++) {
         if (i < nq) {
             float* dst = p.part + (((size_t)m * p.H * p.maps + (size_t)h0 * p.maps + i) * p.splits + split) * (p.vp + 2);
+            if (tid == 0) { dst[0] = sm[i]; dst[1] = sl[i]; }
 #pragma unroll
             for (int c = 0; c < CR; c++) {
                 const int col = tid + c * kRowThreads;
@@ -190,21 +201,24 @@ __global__ void __launch_bounds__(kRowThreads) attention_rows_kernel(const AttnP
 // Adds the key splits of one (row, head) and finishes the head.
 template <typename T>
 __global__ void __launch_bounds__(kRowThreads) attention_merge_kernel(const AttnParams p) {
-    pdl_wait();
     pdl_launch_dependents();
+    pdl_wait();
     __shared__ float red[33];
     __shared__ float sw[2 * kMaxSplits];
     const int h = blockIdx.x, m = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    KeyWalk kw;
+    kw.init(p, m);
+    const int per = kw.per_split(p), ns = (kw.blocks() + per - 1) / per;          // splits that hold something
     const size_t stride = p.vp + 2;
     const float* base = p.part + ((size_t)m * p.H + h) * p.maps * p.splits * stride;
     if (warp < p.maps) {
         const float* b = base + (size_t)warp * p.splits * stride;
-        const float mm = lane < p.splits ? b[lane * stride] : -INFINITY;
-        const float ll = lane < p.splits ? b[lane * stride + 1] : 0.f;
+        const float mm = lane < ns ? b[lane * stride] : -INFINITY;
+        const float ll = lane < ns ? b[lane * stride + 1] : 0.f;
         const float mx = warp_max(mm);
         const float f = mm == -INFINITY ? 0.f : exp2f(mm - mx);
         const float tot = warp_sum(f * ll);
-        if (lane < kMaxSplits) sw[warp * kMaxSplits + lane] = tot > 0.f ? f / tot : 0.f;
+        sw[warp * kMaxSplits + lane] = tot > 0.f ? f / tot : 0.f;
     }
     __syncthreads();
     float ss = 0.f;
@@ -215,11 +229,13 @@ __global__ void __launch_bounds__(kRowThreads) attention_merge_kernel(const Attn
         o[c] = 0.f;
         if (col < p.vdim) {
             float a[2] = {0.f, 0.f};
-            for (int mp = 0; mp < p.maps; mp++)
-                for (int s = 0; s < p.splits; s++) {
-                    const float f = sw[mp * kMaxSplits + s];
-                    if (f != 0.f) a[mp] = fmaf(f, base[((size_t)mp * p.splits + s) * stride + 2 + col], a[mp]);
-                }
+            for (int mp = 0; mp < p.maps; mp++) {
+                const float* src = base + (size_t)mp * p.splits * stride + 2 + col;
+                float x = 0.f;
+#pragma unroll 8
+                for (int s = 0; s < ns; s++) x = fmaf(sw[mp * kMaxSplits + s], src[s * stride], x);
+                a[mp] = x;
+            }
             o[c] = p.maps == 2 ? a[0] - p.lambda * a[1] : a[0];
             ss = fmaf(o[c], o[c], ss);
         }
@@ -258,8 +274,8 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
 
 template <int VT, int MAPS>              // 16-column value tiles, maps per head
 __global__ void __launch_bounds__(128) attention_prompt_kernel(const AttnParams p) {
-    pdl_wait();
     pdl_launch_dependents();
+    pdl_wait();
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int KE = MAPS * p.dp, KP = KE + 8;
     constexpr int VP = VT * 16 + 8;
@@ -471,7 +487,7 @@ void pick_groups(int R, int maps, int* hpg, int* qgroups) {
 template <typename T, int QN>
 int launch_rows(AttnParams& p, cudaStream_t st) {
     const int KP = p.maps * p.dp + 16 / (int)sizeof(T);
-    const size_t smem = (size_t)(QN * p.dp + QN * kKeys + 4 * QN + kKeys) * 4 + (size_t)kKeys * KP * sizeof(T);
+    const size_t smem = (size_t)(QN * p.dp + QN * (kKeys + 4) + 4 * QN + kKeys) * 4 + (size_t)kKeys * (KP + p.vp) * sizeof(T);
     const dim3 grid(p.splits, p.G * p.qgroups, p.M);
     if (p.vdim <= kRowThreads) {
         auto k = attention_rows_kernel<T, QN, 1>;

@@ -50,6 +50,22 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
     return red[32];
 }
 
+// The sums of three values over the CTA at once.  `red` holds 99 floats.
+__device__ __forceinline__ float3 block_sum3(float3 v, float* red) {
+    v.x = warp_sum(v.x); v.y = warp_sum(v.y); v.z = warp_sum(v.z);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+    __syncthreads();
+    if (lane == 0) { red[warp] = v.x; red[33 + warp] = v.y; red[66 + warp] = v.z; }
+    __syncthreads();
+    if (warp < 3) {
+        float t = lane < nw ? red[33 * warp + lane] : 0.f;
+        t = warp_sum(t);
+        if (lane == 0) red[33 * warp + 32] = t;
+    }
+    __syncthreads();
+    return make_float3(red[32], red[65], red[98]);
+}
+
 __host__ __device__ constexpr int round_up(int v, int m) { return (v + m - 1) / m * m; }
 
 // ---------------------------------------------------------------- epilogues of the matrix products
@@ -131,20 +147,44 @@ struct ColumnOut {
             }
         }
     }
-    __device__ __forceinline__ void store(int m, float acc) const {
-        if (base == nullptr) return;
+    __device__ __forceinline__ float finish(float acc, float residual) const {
+        if (op == kOpSilu) return acc * sigmoid_f(acc);
+        if (op == kOpSigmoid) return sigmoid_f(acc);
+        if (op == kOpForget) return (1.0f - p1) * sigmoid_f(-(acc + p0));
+        if (op == kOpResidual) return residual + p0 * acc;
+        if (op == kOpSoftcap && p0 > 0.f) return p0 * tanhf(acc / p0);
+        return acc;
+    }
+    __device__ __forceinline__ float residual(int m) const {
+        float r = *reinterpret_cast<const float*>(base + (long long)m * stride);
+        if (add_base != nullptr) r += *reinterpret_cast<const float*>(add_base + (long long)m * stride);
+        return r;
+    }
+    __device__ __forceinline__ void put(int m, float v) const {
         char* p = base + (long long)m * stride;
-        float v = acc;
-        if (op == kOpSilu) v = acc * sigmoid_f(acc);
-        else if (op == kOpSigmoid) v = sigmoid_f(acc);
-        else if (op == kOpForget) v = (1.0f - p1) * sigmoid_f(-(acc + p0));
-        else if (op == kOpResidual) {
-            v = *reinterpret_cast<float*>(p) + p0 * acc;
-            if (add_base != nullptr) v += *reinterpret_cast<const float*>(add_base + (long long)m * stride);
-        } else if (op == kOpSoftcap && p0 > 0.f) v = p0 * tanhf(acc / p0);
         if (f32) *reinterpret_cast<float*>(p) = v;
         else *reinterpret_cast<T*>(p) = from_f32<T>(v);
         if (half_base != nullptr) half_base[(long long)m * (stride >> 2)] = __float2half_rn(v);
+    }
+    __device__ __forceinline__ void store(int m, float acc) const {
+        if (base == nullptr) return;
+        put(m, finish(acc, op == kOpResidual ? residual(m) : 0.f));
+    }
+    // Rows m0 .. m0 + n - 1 (n <= N): all residual loads before the first store.
+    template <int N>
+    __device__ __forceinline__ void store_rows(int m0, int n, const uint32_t (&acc)[N]) const {
+        if (base == nullptr) return;
+        float r[N];
+#pragma unroll
+        for (int i = 0; i < N; i++) r[i] = 0.f;
+        if (op == kOpResidual) {
+#pragma unroll
+            for (int i = 0; i < N; i++)
+                if (i < n) r[i] = residual(m0 + i);
+        }
+#pragma unroll
+        for (int i = 0; i < N; i++)
+            if (i < n) put(m0 + i, finish(__uint_as_float(acc[i]), r[i]));
     }
 };
 

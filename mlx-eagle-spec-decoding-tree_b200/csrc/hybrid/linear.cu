@@ -230,10 +230,11 @@ __global__ void __launch_bounds__(kThreads) gemm_kernel(const __grid_constant__ 
                     : "r"(taddr + c)
                     : "memory");
                 asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+                if (ks > 1) {
 #pragma unroll
-                for (int i = 0; i < 16; i++) {
-                    if (ks > 1) part[(c + i) * kTileRows + r] = __uint_as_float(v[i]);
-                    else if (tok0 + c + i < p.epi.M) out.store(tok0 + c + i, __uint_as_float(v[i]));
+                    for (int i = 0; i < 16; i++) part[(c + i) * kTileRows + r] = __uint_as_float(v[i]);
+                } else {
+                    out.store_rows<16>(tok0 + c, p.epi.M - tok0 - c, v);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");

@@ -8,13 +8,38 @@ namespace hybrid {
 namespace {
 
 constexpr int kThreads = 256;
-constexpr int kRowsPerCta = 4;       // chain rows of one CTA of the norm + convolution kernel
+constexpr int kRowsPerCta = 8;       // chain rows of one CTA of the norm + convolution kernel
 constexpr int kMaxTaps = B200_HYBRID_MAX_TAPS;
+
+// V (1 or 4) neighbouring channels.
+template <int V> struct Vec { float v[V]; };
+template <int V> __device__ __forceinline__ Vec<V> ld(const float* p) {
+    Vec<V> r;
+    if (V == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        r.v[0] = t.x; r.v[V > 1 ? 1 : 0] = t.y; r.v[V > 1 ? 2 : 0] = t.z; r.v[V > 1 ? 3 : 0] = t.w;
+        return r;
+    }
+    r.v[0] = *p;
+    return r;
+}
+template <int V> __device__ __forceinline__ void st(float* p, const Vec<V>& r) {
+    if (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[V > 1 ? 1 : 0], r.v[V > 1 ? 2 : 0], r.v[V > 1 ? 3 : 0]);
+    else *p = r.v[0];
+}
+template <int V> __device__ __forceinline__ void st(bf16* p, const Vec<V>& r) {
+    if (V == 4) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(r.v[0], r.v[V > 1 ? 1 : 0]), b = __floats2bfloat162_rn(r.v[V > 1 ? 2 : 0], r.v[V > 1 ? 3 : 0]);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+    } else {
+        *p = __float2bfloat16_rn(r.v[0]);
+    }
+}
 
 __global__ void __launch_bounds__(kThreads) embed_kernel(const int* __restrict__ tokens, const bf16* __restrict__ table, int width, int vocab,
                                                          float* __restrict__ x, float* __restrict__ emb) {
-    pdl_wait();
     pdl_launch_dependents();
+    pdl_wait();
     const int m = blockIdx.x;
     const int tok = min(max(tokens[m], 0), vocab - 1);
     for (int c = threadIdx.x; c < width; c += kThreads) {
@@ -24,10 +49,19 @@ __global__ void __launch_bounds__(kThreads) embed_kernel(const int* __restrict__
     }
 }
 
+template <int V>
 __device__ __forceinline__ float row_sumsq_warp(const float* __restrict__ row, int width, int lane) {
-    float s = 0.f;
-    for (int c = lane; c < width; c += 32) { const float v = row[c]; s = fmaf(v, v, s); }
-    return warp_sum(s);
+    float s[V] = {};
+#pragma unroll 8
+    for (int c = lane * V; c < width; c += 32 * V) {
+        const Vec<V> t = ld<V>(row + c);
+#pragma unroll
+        for (int e = 0; e < V; e++) s[e] = fmaf(t.v[e], t.v[e], s[e]);
+    }
+    float r = 0.f;
+#pragma unroll
+    for (int e = 0; e < V; e++) r += s[e];
+    return warp_sum(r);
 }
 
 struct NormConvParams {
@@ -40,30 +74,33 @@ struct NormConvParams {
     const unsigned long long* mask;
     const int* pos;
     int* tail_pos;
-    int M, width, pitch, taps, write_off, tree;
+    int M, width, pitch, write_off;
     float eps;
 };
 
-// h = x / rms(x) * w;  out = h + sum_j conv[j] * (input taps-1-j positions earlier on the row's path).
+// h = x / rms(x) * w;  out = h + sum_j conv[j] * (input TAPS-1-j positions earlier on the row's path).
+// Grid (rows, channel slices); every CTA computes the norms it needs from whole rows.
 // Chain: kRowsPerCta consecutive rows per CTA, the inputs before them recomputed from x or taken from the state.
 // Tree: one row per CTA; its predecessors are its ancestors (set bits of its mask), then the committed inputs.
-template <typename T>
+template <typename T, int TAPS, int V, bool TREE>
 __global__ void __launch_bounds__(kThreads) norm_conv_kernel(const NormConvParams p) {
-    pdl_wait();
     pdl_launch_dependents();
-    __shared__ float s_rstd[kRowsPerCta + kMaxTaps];
+    pdl_wait();
+    constexpr int PREV = TAPS - 1;
+    constexpr int ROWS = TREE ? 1 : kRowsPerCta;
+    __shared__ float s_rstd[ROWS + PREV];
     __shared__ const float* s_src[kMaxTaps];      // tree: predecessor vectors, oldest first
     __shared__ int s_raw[kMaxTaps];               // ... row of this pass whose norm has to be applied (-1: vector as stored)
-    const int W = p.width, prev = p.taps - 1;
+    const int W = p.width;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int r0 = blockIdx.x * ROWS, rows = min(ROWS, p.M - r0);
+    const int self = p.write_off + r0;
     T* out = static_cast<T*>(p.out);
-    if (p.tree) {
-        const int m = blockIdx.x;
-        const int self = p.write_off + m;
+    if (TREE) {
         if (threadIdx.x == 0) {
-            unsigned long long anc = p.mask[m] & ((1ull << self) - 1ull);
+            unsigned long long anc = p.mask[r0] & ((1ull << self) - 1ull);
             int have = 0;
-            for (int j = prev - 1; j >= 0; j--) {
+            for (int j = PREV - 1; j >= 0; j--) {
                 if (anc != 0ull) {
                     const int a = 63 - __clzll((long long)anc);
                     anc &= ~(1ull << a);
@@ -75,121 +112,129 @@ __global__ void __launch_bounds__(kThreads) norm_conv_kernel(const NormConvParam
                     s_src[j] = p.state + (size_t)(j + have) * W;
                 }
             }
-            p.tail_pos[self] = p.pos[m];
+            if (blockIdx.y == 0) p.tail_pos[self] = p.pos[r0];
         }
         __syncthreads();
-        if (warp <= prev) {
-            const int row = warp == prev ? m : s_raw[warp];
-            if (row >= 0) {
-                const float ss = row_sumsq_warp(p.x + (size_t)row * W, W, lane);
-                if (lane == 0) s_rstd[warp] = rsqrtf(ss / (float)W + p.eps);
-            }
-        }
-        __syncthreads();
-        for (int c = threadIdx.x; c < W; c += kThreads) {
-            const float wc = p.w[c];
-            const float h = p.x[(size_t)m * W + c] * s_rstd[prev] * wc;
-            float acc = fmaf(p.conv[(size_t)prev * W + c], h, h);
-            for (int j = 0; j < prev; j++) {
-                float v = s_src[j][c];
-                if (s_raw[j] >= 0) v = v * s_rstd[j] * wc;
-                acc = fmaf(p.conv[(size_t)j * W + c], v, acc);
-            }
-            p.pend[(size_t)self * W + c] = h;
-            out[(size_t)m * p.pitch + c] = from_f32<T>(acc);
-        }
-        return;
     }
-    const int r0 = blockIdx.x * kRowsPerCta, rows = min(kRowsPerCta, p.M - r0);
-    for (int i = warp; i < rows + prev; i += kThreads / 32) {
-        const int row = r0 - prev + i;
+    for (int i = warp; i < rows + PREV; i += kThreads / 32) {
+        const int row = TREE ? (i == PREV ? r0 : s_raw[i]) : r0 - PREV + i;
         if (row >= 0) {
-            const float ss = row_sumsq_warp(p.x + (size_t)row * W, W, lane);
+            const float ss = row_sumsq_warp<V>(p.x + (size_t)row * W, W, lane);
             if (lane == 0) s_rstd[i] = rsqrtf(ss / (float)W + p.eps);
         }
     }
     __syncthreads();
-    for (int c = threadIdx.x; c < W; c += kThreads) {
-        const float wc = p.w[c];
-        float hist[kMaxTaps], cw[kMaxTaps];           // the last entries are the ones in use: hist[kMaxTaps-1] is the newest
+    for (int c = (blockIdx.y * kThreads + threadIdx.x) * V; c < W; c += gridDim.y * kThreads * V) {
+        const Vec<V> wc = ld<V>(p.w + c);
+        Vec<V> hist[TAPS], cw[TAPS];                  // inputs, oldest first
 #pragma unroll
-        for (int j = 0; j < kMaxTaps; j++) {
-            const int k = j - (kMaxTaps - p.taps);    // tap index
-            cw[j] = k >= 0 ? p.conv[(size_t)k * W + c] : 0.f;
-            float v = 0.f;
-            if (k >= 0 && k < prev) {                 // input k - prev positions before row r0 is tap k of row r0 - 0
-                const int row = r0 - prev + k;
-                v = row >= 0 ? p.x[(size_t)row * W + c] * s_rstd[k] * wc : p.state[(size_t)(row + prev) * W + c];
-            }
-            hist[j] = v;
+        for (int k = 0; k < TAPS; k++) cw[k] = ld<V>(p.conv + (size_t)k * W + c);
+#pragma unroll
+        for (int k = 0; k < PREV; k++) {
+            const int row = TREE ? s_raw[k] : r0 - PREV + k;
+            const float* src = TREE ? s_src[k] : (row >= 0 ? p.x + (size_t)row * W : p.state + (size_t)(row + PREV) * W);
+            hist[k] = ld<V>(src + c);
+            if (row >= 0)
+#pragma unroll
+                for (int e = 0; e < V; e++) hist[k].v[e] *= s_rstd[k] * wc.v[e];
         }
-        // shift so that the loop below can push the newest input
 #pragma unroll
-        for (int r = 0; r < kRowsPerCta; r++) {
+        for (int r = 0; r < ROWS; r++) {
             if (r >= rows) break;
             const int m = r0 + r;
-            const float h = p.x[(size_t)m * W + c] * s_rstd[prev + r] * wc;
-            hist[kMaxTaps - 1] = h;
-            float acc = h;
+            Vec<V> h = ld<V>(p.x + (size_t)m * W + c), acc;
 #pragma unroll
-            for (int j = 0; j < kMaxTaps; j++) acc = fmaf(cw[j], hist[j], acc);
-            const int slot = chain_slot(m, p.M);
-            if (slot >= 0 && m >= p.M - prev) p.pend[(size_t)slot * W + c] = h;
-            out[(size_t)m * p.pitch + c] = from_f32<T>(acc);
+            for (int e = 0; e < V; e++) {
+                h.v[e] *= s_rstd[PREV + r] * wc.v[e];
+                acc.v[e] = fmaf(cw[PREV].v[e], h.v[e], h.v[e]);
+            }
 #pragma unroll
-            for (int j = 0; j + 1 < kMaxTaps; j++) hist[j] = hist[j + 1];
+            for (int k = 0; k < PREV; k++)
+#pragma unroll
+                for (int e = 0; e < V; e++) acc.v[e] = fmaf(cw[k].v[e], hist[k].v[e], acc.v[e]);
+            if (TREE) st<V>(p.pend + (size_t)self * W + c, h);
+            else if (m >= p.M - PREV) st<V>(p.pend + (size_t)chain_slot(m, p.M) * W + c, h);
+            st<V>(out + (size_t)m * p.pitch + c, acc);
+#pragma unroll
+            for (int k = 0; k + 1 < PREV; k++) hist[k] = hist[k + 1];
+            if (PREV > 0) hist[PREV > 0 ? PREV - 1 : 0] = h;
         }
     }
 }
 
-template <typename T>
-__global__ void __launch_bounds__(kThreads) norm_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ out,
-                                                        const int* __restrict__ rows, const int* __restrict__ row_index, int gather,
-                                                        int width, int pitch, float eps) {
-    pdl_wait();
+template <typename T, int V>
+__global__ void __launch_bounds__(1024) norm_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ out,
+                                                    const int* __restrict__ rows, const int* __restrict__ row_index, int gather, int width,
+                                                    int pitch, float eps) {
     pdl_launch_dependents();
+    pdl_wait();
     __shared__ float red[33];
     int src = blockIdx.x;
     if (gather) src = rows != nullptr ? rows[src] : (row_index != nullptr ? row_index[0] + src : src);
     const float* xr = x + (size_t)src * width;
     float ss = 0.f;
-    for (int c = threadIdx.x; c < width; c += kThreads) { const float v = xr[c]; ss = fmaf(v, v, ss); }
+#pragma unroll 4
+    for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+        const Vec<V> t = ld<V>(xr + c);
+#pragma unroll
+        for (int e = 0; e < V; e++) ss = fmaf(t.v[e], t.v[e], ss);
+    }
     ss = block_sum(ss, red);
     const float rstd = rsqrtf(ss / (float)width + eps);
     T* o = out + (size_t)blockIdx.x * pitch;
-    for (int c = threadIdx.x; c < width; c += kThreads) o[c] = from_f32<T>(xr[c] * rstd * w[c]);
+#pragma unroll 4
+    for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+        Vec<V> t = ld<V>(xr + c);
+        const Vec<V> g = ld<V>(w + c);
+#pragma unroll
+        for (int e = 0; e < V; e++) t.v[e] *= rstd * g.v[e];
+        st<V>(o + c, t);
+    }
 }
 
-// a N(z) + b N(z^2) + c N(z^3) + e, N: over the root mean square of the row.
+// a N(z) + b N(z^2) + c N(z^3) + e, N: over the root mean square of the row.  16 bytes per thread and step; the padding of
+// a row (zeros or finite leftovers that meet zero weights) is read but not counted.
 template <typename T>
-__global__ void __launch_bounds__(kThreads) polynorm_kernel(const T* __restrict__ z, T* __restrict__ out, int width, int pitch, float a, float b,
-                                                            float c, float e, float eps) {
-    pdl_wait();
+__global__ void __launch_bounds__(1024) polynorm_kernel(const T* __restrict__ z, T* __restrict__ out, int width, int pitch, float a, float b,
+                                                        float c, float e, float eps) {
     pdl_launch_dependents();
-    __shared__ float red[33];
+    pdl_wait();
+    constexpr int VE = 16 / (int)sizeof(T);
+    __shared__ float red[99];
     const T* zr = z + (size_t)blockIdx.x * pitch;
-    float s1 = 0.f, s2 = 0.f, s3 = 0.f;
-    for (int i = threadIdx.x; i < width; i += kThreads) {
-        const float v = to_f32<T>(zr[i]), q = v * v, u = q * v;
-        s1 += q;
-        s2 = fmaf(q, q, s2);
-        s3 = fmaf(u, u, s3);
+    float3 s = make_float3(0.f, 0.f, 0.f);
+#pragma unroll 2
+    for (int i = threadIdx.x * VE; i < width; i += blockDim.x * VE) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(zr + i);
+        const T* t = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+        for (int k = 0; k < VE; k++) {
+            const float v = i + k < width ? to_f32<T>(t[k]) : 0.f, q = v * v, u = q * v;
+            s.x += q;
+            s.y = fmaf(q, q, s.y);
+            s.z = fmaf(u, u, s.z);
+        }
     }
-    s1 = block_sum(s1, red);
-    s2 = block_sum(s2, red);
-    s3 = block_sum(s3, red);
+    s = block_sum3(s, red);
     const float n = (float)width;
-    const float ka = a * rsqrtf(s1 / n + eps), kb = b * rsqrtf(s2 / n + eps), kc = c * rsqrtf(s3 / n + eps);
+    const float ka = a * rsqrtf(s.x / n + eps), kb = b * rsqrtf(s.y / n + eps), kc = c * rsqrtf(s.z / n + eps);
     T* o = out + (size_t)blockIdx.x * pitch;
-    for (int i = threadIdx.x; i < width; i += kThreads) {
-        const float v = to_f32<T>(zr[i]);
-        o[i] = from_f32<T>(fmaf(v, fmaf(v, fmaf(v, kc, kb), ka), e));
+#pragma unroll 2
+    for (int i = threadIdx.x * VE; i < width; i += blockDim.x * VE) {
+        uint4 raw = *reinterpret_cast<const uint4*>(zr + i);
+        T* t = reinterpret_cast<T*>(&raw);
+#pragma unroll
+        for (int k = 0; k < VE; k++) {
+            const float v = to_f32<T>(t[k]);
+            t[k] = from_f32<T>(i + k < width ? fmaf(v, fmaf(v, fmaf(v, kc, kb), ka), e) : 0.f);
+        }
+        *reinterpret_cast<uint4*>(o + i) = raw;
     }
 }
 
 __global__ void add_kernel(float* __restrict__ x, const float* __restrict__ y, size_t n) {
-    pdl_wait();
     pdl_launch_dependents();
+    pdl_wait();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i < n) x[i] += y[i];
 }
@@ -202,6 +247,59 @@ int launch_embed(const b200_hybrid_model& m, const b200_hybrid_pass& p, cudaStre
     return check_launch();
 }
 
+namespace {
+
+template <typename T, int TAPS, int V>
+void launch_norm_conv_v(const NormConvParams& q, int tree, cudaStream_t st) {
+    const int all = (q.width + kThreads * V - 1) / (kThreads * V);
+    const int slices = q.M <= 32 ? all : 1;          // many rows: a CTA takes whole rows, or it would read them once per slice
+    if (tree) launch_kernel(norm_conv_kernel<T, TAPS, V, true>, dim3(q.M, slices), dim3(kThreads), 0, st, q);
+    else launch_kernel(norm_conv_kernel<T, TAPS, V, false>, dim3((q.M + kRowsPerCta - 1) / kRowsPerCta, slices), dim3(kThreads), 0, st, q);
+}
+
+template <typename T, int TAPS>
+int launch_norm_conv_t(const NormConvParams& q, int taps, int tree, cudaStream_t st) {
+    if constexpr (TAPS > kMaxTaps) {
+        return B200_ELIMIT;
+    } else {
+        if (taps != TAPS) return launch_norm_conv_t<T, TAPS + 1>(q, taps, tree, st);
+        if (q.width % 4 == 0) launch_norm_conv_v<T, TAPS, 4>(q, tree, st);
+        else launch_norm_conv_v<T, TAPS, 1>(q, tree, st);
+        return check_launch();
+    }
+}
+
+// Threads of a CTA that works on one row: more when there are few rows.
+int row_threads(int rows, int units) {
+    const int most = rows < 148 ? 1024 : 256;
+    const int t = round_up(units, 32);
+    return t < 128 ? 128 : (t < most ? t : most);    // (block_sum3 needs three warps)
+}
+
+template <typename T>
+int launch_norm_t(const b200_hybrid_model& m, const float* w, const b200_hybrid_pass& p, int gather, int rows, cudaStream_t st) {
+    const int pitch = round_up(m.width, 64);
+    const float* x = m.x;
+    T* out = static_cast<T*>(m.hb);
+    if (m.width % 4 == 0)
+        launch_kernel(norm_kernel<T, 4>, dim3(rows), dim3(row_threads(rows, m.width / 4)), 0, st, x, w, out, p.out_rows, p.row_index, gather,
+                      m.width, pitch, m.eps);
+    else
+        launch_kernel(norm_kernel<T, 1>, dim3(rows), dim3(row_threads(rows, m.width)), 0, st, x, w, out, p.out_rows, p.row_index, gather, m.width,
+                      pitch, m.eps);
+    return check_launch();
+}
+
+template <typename T>
+int launch_polynorm_t(const b200_hybrid_model& m, const b200_hybrid_layer& l, int rows, cudaStream_t st) {
+    const int VE = 16 / (int)sizeof(T);
+    launch_kernel(polynorm_kernel<T>, dim3(rows), dim3(row_threads(rows, (l.ff + VE - 1) / VE)), 0, st, static_cast<const T*>(m.zb),
+                  static_cast<T*>(m.zab), l.ff, round_up(l.ff, 64), l.act[0], l.act[1], l.act[2], l.act[3], m.eps);
+    return check_launch();
+}
+
+}  // namespace
+
 int launch_norm_conv(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_run& r, const b200_hybrid_pass& p,
                      cudaStream_t st) {
     NormConvParams q{};
@@ -209,34 +307,17 @@ int launch_norm_conv(const b200_hybrid_model& m, const b200_hybrid_layer& l, con
     q.state = reinterpret_cast<const float*>(static_cast<const char*>(p.cache) + r.conv_off);
     q.pend = reinterpret_cast<float*>(static_cast<char*>(m.pending) + r.pend_h);
     q.out = m.hb; q.mask = p.mask; q.pos = p.pos; q.tail_pos = p.tail_pos;
-    q.M = p.M; q.width = m.width; q.pitch = round_up(m.width, 64); q.taps = l.taps; q.write_off = p.write_off; q.tree = p.tree;
+    q.M = p.M; q.width = m.width; q.pitch = round_up(m.width, 64); q.write_off = p.write_off;
     q.eps = m.eps;
-    const int grid = p.tree ? p.M : (p.M + kRowsPerCta - 1) / kRowsPerCta;
-    if (m.act_type == B200_ACT_F32) launch_kernel(norm_conv_kernel<float>, dim3(grid), dim3(kThreads), 0, st, q);
-    else launch_kernel(norm_conv_kernel<bf16>, dim3(grid), dim3(kThreads), 0, st, q);
-    return check_launch();
+    return m.act_type == B200_ACT_F32 ? launch_norm_conv_t<float, 1>(q, l.taps, p.tree, st) : launch_norm_conv_t<bf16, 1>(q, l.taps, p.tree, st);
 }
 
 int launch_norm(const b200_hybrid_model& m, const float* w, const b200_hybrid_pass& p, bool gather, int rows, cudaStream_t st) {
-    const int pitch = round_up(m.width, 64), g = gather ? 1 : 0;
-    if (m.act_type == B200_ACT_F32)
-        launch_kernel(norm_kernel<float>, dim3(rows), dim3(kThreads), 0, st, static_cast<const float*>(m.x), w, static_cast<float*>(m.hb),
-                      p.out_rows, p.row_index, g, m.width, pitch, m.eps);
-    else
-        launch_kernel(norm_kernel<bf16>, dim3(rows), dim3(kThreads), 0, st, static_cast<const float*>(m.x), w, static_cast<bf16*>(m.hb),
-                      p.out_rows, p.row_index, g, m.width, pitch, m.eps);
-    return check_launch();
+    return m.act_type == B200_ACT_F32 ? launch_norm_t<float>(m, w, p, gather ? 1 : 0, rows, st) : launch_norm_t<bf16>(m, w, p, gather ? 1 : 0, rows, st);
 }
 
 int launch_polynorm(const b200_hybrid_model& m, const b200_hybrid_layer& l, int rows, cudaStream_t st) {
-    const int pitch = round_up(l.ff, 64);
-    if (m.act_type == B200_ACT_F32)
-        launch_kernel(polynorm_kernel<float>, dim3(rows), dim3(kThreads), 0, st, static_cast<const float*>(m.zb), static_cast<float*>(m.zab),
-                      l.ff, pitch, l.act[0], l.act[1], l.act[2], l.act[3], m.eps);
-    else
-        launch_kernel(polynorm_kernel<bf16>, dim3(rows), dim3(kThreads), 0, st, static_cast<const bf16*>(m.zb), static_cast<bf16*>(m.zab),
-                      l.ff, pitch, l.act[0], l.act[1], l.act[2], l.act[3], m.eps);
-    return check_launch();
+    return m.act_type == B200_ACT_F32 ? launch_polynorm_t<float>(m, l, rows, st) : launch_polynorm_t<bf16>(m, l, rows, st);
 }
 
 int launch_add(float* x, const float* y, size_t n, cudaStream_t st) {

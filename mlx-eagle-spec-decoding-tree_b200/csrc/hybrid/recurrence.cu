@@ -18,11 +18,29 @@ namespace {
 constexpr int kWarps = 8;
 constexpr int kMaxDim = 256;
 
+// Two fp32 values in one register pair: packed multiply-adds, each half rounded as a single one.
+__device__ __forceinline__ unsigned long long pack2(float a, float b) {
+    unsigned long long r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float2 unpack2(unsigned long long v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+    unsigned long long r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+constexpr unsigned long long kMinusOne2 = 0xbf800000bf800000ull;
+
 template <typename T, int DR, int TB>    // state rows of a warp, tokens of a block
 __global__ void __launch_bounds__(kWarps * 32) scan_kernel(const T* __restrict__ q, const float* __restrict__ gf, const T* __restrict__ v,
                                                            float* __restrict__ state, float* __restrict__ o, int M, int H, int d, int dv) {
-    pdl_wait();
     pdl_launch_dependents();
+    pdl_wait();
     constexpr int D = kWarps * DR;
     constexpr int PER = TB * D / (kWarps * 32), PERV = (TB * 32 + kWarps * 32 - 1) / (kWarps * 32);
     __shared__ __align__(16) float sg[TB][D];
@@ -31,10 +49,13 @@ __global__ void __launch_bounds__(kWarps * 32) scan_kernel(const T* __restrict__
     __shared__ float part[kWarps][TB][32];
     const int h = blockIdx.y, c0 = blockIdx.x * 32, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int col = c0 + lane;
-    float S[DR];
+    unsigned long long S[DR / 2];        // two neighbouring state rows each
     float* sbase = state + ((size_t)h * d + warp * DR) * dv + col;
 #pragma unroll
-    for (int r = 0; r < DR; r++) S[r] = (warp * DR + r < d && col < dv) ? sbase[(size_t)r * dv] : 0.f;
+    for (int r = 0; r < DR; r += 2) {
+        const int i = warp * DR + r;
+        S[r / 2] = pack2(i < d && col < dv ? sbase[(size_t)r * dv] : 0.f, i + 1 < d && col < dv ? sbase[(size_t)(r + 1) * dv] : 0.f);
+    }
     float pg[PER], pq[PER], pv[PERV];
     auto fetch = [&](int t0) {
 #pragma unroll
@@ -67,24 +88,27 @@ __global__ void __launch_bounds__(kWarps * 32) scan_kernel(const T* __restrict__
         __syncthreads();
         if (t0 + TB < M) fetch(t0 + TB);
         const int nt = min(TB, M - t0);
-#pragma unroll 2
-        for (int t = 0; t < nt; t++) {
+        auto token = [&](int t) {
             const float vt = sv[t][lane];
-            float a0 = 0.f, a1 = 0.f;
+            const unsigned long long v2 = pack2(vt, vt);
+            unsigned long long a0 = 0ull, a1 = 0ull;
 #pragma unroll
             for (int r = 0; r < DR; r += 4) {
-                const float4 g4 = *reinterpret_cast<const float4*>(&sg[t][warp * DR + r]);
-                const float4 q4 = *reinterpret_cast<const float4*>(&sq[t][warp * DR + r]);
-                S[r] = fmaf(g4.x, vt - S[r], S[r]);
-                S[r + 1] = fmaf(g4.y, vt - S[r + 1], S[r + 1]);
-                S[r + 2] = fmaf(g4.z, vt - S[r + 2], S[r + 2]);
-                S[r + 3] = fmaf(g4.w, vt - S[r + 3], S[r + 3]);
-                a0 = fmaf(q4.x, S[r], a0);
-                a1 = fmaf(q4.y, S[r + 1], a1);
-                a0 = fmaf(q4.z, S[r + 2], a0);
-                a1 = fmaf(q4.w, S[r + 3], a1);
+                const ulonglong2 g4 = *reinterpret_cast<const ulonglong2*>(&sg[t][warp * DR + r]);
+                const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(&sq[t][warp * DR + r]);
+                S[r / 2] = fma2(g4.x, fma2(S[r / 2], kMinusOne2, v2), S[r / 2]);
+                S[r / 2 + 1] = fma2(g4.y, fma2(S[r / 2 + 1], kMinusOne2, v2), S[r / 2 + 1]);
+                a0 = fma2(q4.x, S[r / 2], a0);
+                a1 = fma2(q4.y, S[r / 2 + 1], a1);
             }
-            part[warp][t][lane] = a0 + a1;
+            const float2 x = unpack2(a0), y = unpack2(a1);
+            part[warp][t][lane] = (x.x + x.y) + (y.x + y.y);
+        };
+        if (nt == TB) {
+#pragma unroll 4
+            for (int t = 0; t < TB; t++) token(t);
+        } else {
+            for (int t = 0; t < nt; t++) token(t);
         }
         __syncthreads();
         for (int e = tid; e < nt * 32; e += kWarps * 32) {
@@ -96,16 +120,20 @@ __global__ void __launch_bounds__(kWarps * 32) scan_kernel(const T* __restrict__
         }
     }
 #pragma unroll
-    for (int r = 0; r < DR; r++)
-        if (warp * DR + r < d && col < dv) sbase[(size_t)r * dv] = S[r];
+    for (int r = 0; r < DR; r += 2) {
+        const int i = warp * DR + r;
+        const float2 x = unpack2(S[r / 2]);
+        if (i < d && col < dv) sbase[(size_t)r * dv] = x.x;
+        if (i + 1 < d && col < dv) sbase[(size_t)(r + 1) * dv] = x.y;
+    }
 }
 
 template <typename T>
 __global__ void __launch_bounds__(128) tree_kernel(const T* __restrict__ q, const float* __restrict__ pend_g, const T* __restrict__ pend_v,
                                                    const float* __restrict__ state, const unsigned long long* __restrict__ mask,
                                                    float* __restrict__ o, int H, int d, int dv) {
-    pdl_wait();
     pdl_launch_dependents();
+    pdl_wait();
     __shared__ float sw[B200_HYBRID_PENDING][4];
     __shared__ float sqs[kMaxDim];
     const int h = blockIdx.x, m = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -153,8 +181,8 @@ __global__ void __launch_bounds__(128) tree_kernel(const T* __restrict__ q, cons
 template <typename T>
 __global__ void __launch_bounds__(128) head_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, T* __restrict__ out, int M, int H,
                                                         int dv, int pitch, float eps) {
-    pdl_wait();
     pdl_launch_dependents();
+    pdl_wait();
     const int unit = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (unit >= M * H) return;
     const int m = unit / H, h = unit - m * H;
@@ -179,8 +207,8 @@ struct CommitParams {
 
 template <typename T>
 __global__ void __launch_bounds__(256) commit_kernel(const CommitParams p) {
-    pdl_wait();
     pdl_launch_dependents();
+    pdl_wait();
     __shared__ int srow[B200_HYBRID_PENDING];
     const b200_hybrid_run& r = p.runs[blockIdx.x];
     const b200_hybrid_layer& l = p.layers[r.layer];
