@@ -25,7 +25,8 @@ inline int check_launch() {
 
 // Programmatic dependent launch: every kernel of this library may start while its predecessor in
 // the stream is still draining; it must execute pdl_wait() before it reads anything an earlier
-// kernel wrote and before its first global write.  0 disables the launch attribute.
+// kernel wrote and before its first global write.  Pointers to such data carry no __restrict__: the compiler would take
+// it for constant and could move loads across the wait.  0 disables the launch attribute.
 extern int g_use_pdl;
 
 // Poll limit of the device-side waits on other CTAs or other GPUs (grid barrier, all-GPU barrier, argmax

@@ -282,7 +282,7 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const AttnParams 
     bf16* sq = reinterpret_cast<bf16*>(smem_raw);                        // [64][KP]
     bf16* sk = sq + kQRows * KP;                                         // [2][64][KP]
     bf16* sv = sk + 2 * kKeys * KP;                                      // [2][64][VP]
-    const int h = blockIdx.x, r0 = blockIdx.y * kQRows, g = h / (p.H / p.G);
+    const int h = blockIdx.x, r0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * kQRows, g = h / (p.H / p.G);   // longest rows first
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, t = lane & 3;
     const int base_pos = p.prefix[0], qpos0 = base_pos + r0, qlast = base_pos + min(p.M, r0 + kQRows) - 1;
     const bf16* kbase = static_cast<const bf16*>(p.kc) + (size_t)g * p.cap * KE;

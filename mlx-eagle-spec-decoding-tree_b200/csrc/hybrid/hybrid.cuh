@@ -13,6 +13,9 @@
 namespace b200 {
 namespace hybrid {
 
+// (Kernel parameters carry no __restrict__: the compiler would take what earlier kernels wrote for constant and could move
+// its loads across the grid-dependency wait.)
+
 using bf16 = __nv_bfloat16;
 
 template <typename T> __device__ __forceinline__ float to_f32(T v);
@@ -170,21 +173,49 @@ struct ColumnOut {
         if (base == nullptr) return;
         put(m, finish(acc, op == kOpResidual ? residual(m) : 0.f));
     }
-    // Rows m0 .. m0 + n - 1 (n <= N): all residual loads before the first store.
+    template <int OP, bool F32, int N>
+    __device__ __forceinline__ void rows_of(int m0, int n, const uint32_t (&acc)[N]) const {
+        char* p = base + (long long)m0 * stride;
+        float r[N];
+        if (OP == kOpResidual) {                     // all loads before the first store
+#pragma unroll
+            for (int i = 0; i < N; i++) r[i] = i < n ? *reinterpret_cast<const float*>(p + i * stride) : 0.f;
+            if (add_base != nullptr) {
+                const char* q = add_base + (long long)m0 * stride;
+                float e[N];
+#pragma unroll
+                for (int i = 0; i < N; i++) e[i] = i < n ? *reinterpret_cast<const float*>(q + i * stride) : 0.f;
+#pragma unroll
+                for (int i = 0; i < N; i++) r[i] += e[i];
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < N; i++) {
+            float v = __uint_as_float(acc[i]);
+            if (OP == kOpSilu) v = v * sigmoid_f(v);
+            else if (OP == kOpSigmoid) v = sigmoid_f(v);
+            else if (OP == kOpForget) v = (1.0f - p1) * sigmoid_f(-(v + p0));
+            else if (OP == kOpResidual) v = r[i] + p0 * v;
+            else if (OP == kOpSoftcap) v = p0 > 0.f ? p0 * tanhf(v / p0) : v;
+            if (i < n) {
+                if (F32) *reinterpret_cast<float*>(p + i * stride) = v;
+                else *reinterpret_cast<T*>(p + i * stride) = from_f32<T>(v);
+                if (OP == kOpSoftcap && half_base != nullptr) half_base[(long long)(m0 + i) * (stride >> 2)] = __float2half_rn(v);
+            }
+        }
+    }
+    // Rows m0 .. m0 + n - 1, n clipped to N: one branch on the operation, straight code for the rows.
     template <int N>
     __device__ __forceinline__ void store_rows(int m0, int n, const uint32_t (&acc)[N]) const {
         if (base == nullptr) return;
-        float r[N];
-#pragma unroll
-        for (int i = 0; i < N; i++) r[i] = 0.f;
-        if (op == kOpResidual) {
-#pragma unroll
-            for (int i = 0; i < N; i++)
-                if (i < n) r[i] = residual(m0 + i);
+        switch (op) {
+            case kOpNone: if (f32) rows_of<kOpNone, true>(m0, n, acc); else rows_of<kOpNone, false>(m0, n, acc); break;
+            case kOpSilu: rows_of<kOpSilu, false>(m0, n, acc); break;
+            case kOpSigmoid: rows_of<kOpSigmoid, false>(m0, n, acc); break;
+            case kOpForget: rows_of<kOpForget, true>(m0, n, acc); break;
+            case kOpResidual: rows_of<kOpResidual, true>(m0, n, acc); break;
+            default: rows_of<kOpSoftcap, true>(m0, n, acc); break;
         }
-#pragma unroll
-        for (int i = 0; i < N; i++)
-            if (i < n) put(m0 + i, finish(__uint_as_float(acc[i]), r[i]));
     }
 };
 

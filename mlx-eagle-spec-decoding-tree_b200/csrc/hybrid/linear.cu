@@ -28,6 +28,7 @@ constexpr int kTileK = 64;                        // 128 bytes of bf16: one swiz
 constexpr int kWBytes = kTileRows * kTileK * 2;
 constexpr int kEpiWarps = 4;
 constexpr int kThreads = (kEpiWarps + 2) * 32;    // + TMA producer warp + MMA warp
+constexpr int kMaxSplit = 8;                      // CTAs of a cluster
 constexpr uint32_t kPolls = 1u << 22;
 constexpr uint32_t kPollNs = 64u;
 
@@ -35,7 +36,8 @@ template <int NT>
 struct Geo {
     static constexpr int XBYTES = NT * kTileK * 2;
     static constexpr int STAGE = kWBytes + XBYTES;
-    static constexpr int STAGES = NT <= 32 ? 5 : (NT <= 128 ? (NT == 64 ? 4 : 6) : 4);
+    static constexpr int STAGES = NT == 16 ? 6 : (NT == 32 ? 5 : (NT == 128 ? 6 : 4));
+    static constexpr int PER_SM = NT <= 64 ? 2 : 1;        // resident CTAs the shared memory allows
     static constexpr int NACC = NT >= 128 ? 2 : 1;
     static constexpr int ACC_COLS = NT < 32 ? 32 : NT;
     static constexpr int TMEM_COLS = ACC_COLS * NACC;
@@ -80,7 +82,7 @@ __device__ __forceinline__ float ld_cluster_f32(uint32_t saddr, uint32_t rank) {
 }
 
 template <int NT>
-__global__ void __launch_bounds__(kThreads) gemm_kernel(const __grid_constant__ GemmParams p) {
+__global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const __grid_constant__ GemmParams p) {
     using G = Geo<NT>;
     extern __shared__ unsigned char smem_raw[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -250,18 +252,21 @@ __global__ void __launch_bounds__(kThreads) gemm_kernel(const __grid_constant__ 
         __syncthreads();
         cluster_sync_all();
         if (tile0 < tiles && !*abort_flag) {
-            const int share = kTileRows / ks;                       // 16 .. 64 rows
+            const int r0 = kTileRows * (int)rank / ks, share = kTileRows * ((int)rank + 1) / ks - r0;
+            const int tok0 = (tile0 % p.ttiles) * NT, ntok = min(NT, p.epi.M - tok0);
             const uint32_t part = smem_u32(smem);
-            for (int i = threadIdx.x; i < share * ((kThreads) / share); i += kThreads) {
-                const int r = (int)rank * share + i % share;
+            for (int i = threadIdx.x; i < share * ntok; i += kThreads) {
+                const int c = i / share, r = r0 + i - c * share;
                 ColumnOut<bf16> out;
                 out.init(p.epi, (tile0 / p.ttiles) * kTileRows + r);
-                const int tok0 = (tile0 % p.ttiles) * NT;
-                for (int c = i / share; c < NT && tok0 + c < p.epi.M; c += kThreads / share) {
-                    float a = 0.f;
-                    for (int q = 0; q < ks; q++) a += ld_cluster_f32(part + (uint32_t)((c * kTileRows + r) * 4), (uint32_t)q);
-                    out.store(tok0 + c, a);
-                }
+                float v[kMaxSplit];
+#pragma unroll
+                for (int q = 0; q < kMaxSplit; q++)
+                    v[q] = q < ks ? ld_cluster_f32(part + (uint32_t)((c * kTileRows + r) * 4), (uint32_t)q) : 0.f;
+                float a = 0.f;
+#pragma unroll
+                for (int q = 0; q < kMaxSplit; q++) a += v[q];
+                out.store(tok0 + c, a);
             }
         }
         cluster_sync_all();                                        // no CTA leaves while its shared memory is read
@@ -332,10 +337,15 @@ int launch_gemm(const b200_linear& lin, const void* x, int x_rows, const Epi& ep
     p.error = error;
     p.ksplit = 1;
     const int sms = sm_count(), tiles = p.ntiles * p.ttiles;
-    const int slots = sms * (NT <= 64 ? 2 : 1);
     if (NT <= 128) {
-        // split K while the CTAs fit the device at once and every slice keeps at least two K blocks
-        while (p.ksplit < 8 && tiles * p.ksplit * 2 <= slots && p.kblocks >= 4 * p.ksplit) p.ksplit *= 2;
+        // Cut K so that the tiles' slices cover the SMs evenly: one CTA per SM where that uses most of them (its neighbour
+        // in the stream can then sit beside it and fetch weights ahead), else two.
+        float best = 0.f;
+        for (int k = 1; k <= kMaxSplit && k * 2 <= p.kblocks && tiles * k <= sms * G::PER_SM; k++) {
+            const int per_sm = (tiles * k + sms - 1) / sms;
+            const float used = (float)(tiles * k) / (float)(sms * per_sm) - (per_sm > 1 ? 0.1f : 0.f);
+            if (used > best) { best = used; p.ksplit = k; }
+        }
     }
     int grid = tiles * p.ksplit;
     if (p.ksplit == 1 && G::NACC > 1 && grid > sms) grid = sms;     // persistent
@@ -366,7 +376,7 @@ int launch_gemm(const b200_linear& lin, const void* x, int x_rows, const Epi& ep
 
 // ---------------------------------------------------------------- fp32 activations
 // Few rows: one warp per output column, the rows in groups of 8.
-__global__ void __launch_bounds__(256) linear_f32_rows_kernel(const bf16* __restrict__ w, const float* __restrict__ x, int N, int pitch,
+__global__ void __launch_bounds__(256) linear_f32_rows_kernel(const bf16* w, const float* x, int N, int pitch,
                                                               const __grid_constant__ Epi epi) {
     pdl_wait();
     pdl_launch_dependents();
@@ -396,7 +406,7 @@ __global__ void __launch_bounds__(256) linear_f32_rows_kernel(const bf16* __rest
 }
 
 // Many rows: 64 columns x 64 rows per CTA, 4 x 4 per thread.
-__global__ void __launch_bounds__(256) linear_f32_tile_kernel(const bf16* __restrict__ w, const float* __restrict__ x, int N, int pitch,
+__global__ void __launch_bounds__(256) linear_f32_tile_kernel(const bf16* w, const float* x, int N, int pitch,
                                                               const __grid_constant__ Epi epi) {
     pdl_wait();
     pdl_launch_dependents();

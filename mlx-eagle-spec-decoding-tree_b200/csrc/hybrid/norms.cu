@@ -36,8 +36,8 @@ template <int V> __device__ __forceinline__ void st(bf16* p, const Vec<V>& r) {
     }
 }
 
-__global__ void __launch_bounds__(kThreads) embed_kernel(const int* __restrict__ tokens, const bf16* __restrict__ table, int width, int vocab,
-                                                         float* __restrict__ x, float* __restrict__ emb) {
+__global__ void __launch_bounds__(kThreads) embed_kernel(const int* tokens, const bf16* table, int width, int vocab,
+                                                         float* x, float* emb) {
     pdl_launch_dependents();
     pdl_wait();
     const int m = blockIdx.x;
@@ -50,7 +50,7 @@ __global__ void __launch_bounds__(kThreads) embed_kernel(const int* __restrict__
 }
 
 template <int V>
-__device__ __forceinline__ float row_sumsq_warp(const float* __restrict__ row, int width, int lane) {
+__device__ __forceinline__ float row_sumsq_warp(const float* row, int width, int lane) {
     float s[V] = {};
 #pragma unroll 8
     for (int c = lane * V; c < width; c += 32 * V) {
@@ -163,8 +163,8 @@ __global__ void __launch_bounds__(kThreads) norm_conv_kernel(const NormConvParam
 }
 
 template <typename T, int V>
-__global__ void __launch_bounds__(1024) norm_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ out,
-                                                    const int* __restrict__ rows, const int* __restrict__ row_index, int gather, int width,
+__global__ void __launch_bounds__(1024) norm_kernel(const float* x, const float* w, T* out,
+                                                    const int* rows, const int* row_index, int gather, int width,
                                                     int pitch, float eps) {
     pdl_launch_dependents();
     pdl_wait();
@@ -195,7 +195,7 @@ __global__ void __launch_bounds__(1024) norm_kernel(const float* __restrict__ x,
 // a N(z) + b N(z^2) + c N(z^3) + e, N: over the root mean square of the row.  16 bytes per thread and step; the padding of
 // a row (zeros or finite leftovers that meet zero weights) is read but not counted.
 template <typename T>
-__global__ void __launch_bounds__(1024) polynorm_kernel(const T* __restrict__ z, T* __restrict__ out, int width, int pitch, float a, float b,
+__global__ void __launch_bounds__(1024) polynorm_kernel(const T* z, T* out, int width, int pitch, float a, float b,
                                                         float c, float e, float eps) {
     pdl_launch_dependents();
     pdl_wait();
@@ -232,7 +232,7 @@ __global__ void __launch_bounds__(1024) polynorm_kernel(const T* __restrict__ z,
     }
 }
 
-__global__ void add_kernel(float* __restrict__ x, const float* __restrict__ y, size_t n) {
+__global__ void add_kernel(float* x, const float* y, size_t n) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;

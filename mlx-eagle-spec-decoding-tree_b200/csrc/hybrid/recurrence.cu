@@ -2,20 +2,23 @@
 //     S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T   computed as   S += (1 - f) (v - S),      o_t = S_t^T q_t,
 // all in fp32, the state [heads][dim][vdim] carried in the request's cache.
 //
-//   scan_kernel    chain passes, any number of rows: CTA = (head, 32 state columns), warp = a slice of the state's rows,
-//                  lane = column; the slice lives in registers, tokens come in blocks through shared memory, the warps'
-//                  parts of an output are added once per block.  The new state is written back.
+//   scan_kernel    chain passes, any number of rows: CTA = (head, 32 state columns), warp = 4 columns, lane = a slice of
+//                  the state's rows; the slice lives in registers (packed pairs of rows), tokens come in blocks through
+//                  shared memory, the lanes' parts of the outputs are added for 8 tokens at once.  The new state is
+//                  written back.
 //   tree_kernel    tree passes: nothing may change the state yet.  Row m's output is written out along its path:
 //                  o = S_0^T (q prod f) + sum over the path's rows a of (q . (1 - f_a) prod of the later f) v_a.
 //   commit_kernel  advances convolution inputs, states and K/V rows over accepted rows, for every layer run at once.
 //   head_norm      per-head RMS norm of the outputs with the head weight, to the activation type.
 #include "hybrid.cuh"
+#include "../pipeline.cuh"
 
 namespace b200 {
 namespace hybrid {
 namespace {
 
 constexpr int kWarps = 8;
+constexpr int kLaneCols = 4;         // state columns of a warp of the scan
 constexpr int kMaxDim = 256;
 
 // Two fp32 values in one register pair: packed multiply-adds, each half rounded as a single one.
@@ -36,102 +39,140 @@ __device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigne
 }
 constexpr unsigned long long kMinusOne2 = 0xbf800000bf800000ull;
 
-template <typename T, int DR, int TB>    // state rows of a warp, tokens of a block
-__global__ void __launch_bounds__(kWarps * 32) scan_kernel(const T* __restrict__ q, const float* __restrict__ gf, const T* __restrict__ v,
-                                                           float* __restrict__ state, float* __restrict__ o, int M, int H, int d, int dv) {
-    pdl_launch_dependents();
-    pdl_wait();
-    constexpr int D = kWarps * DR;
-    constexpr int PER = TB * D / (kWarps * 32), PERV = (TB * 32 + kWarps * 32 - 1) / (kWarps * 32);
-    __shared__ __align__(16) float sg[TB][D];
-    __shared__ __align__(16) float sq[TB][D];
-    __shared__ float sv[TB][32];
-    __shared__ float part[kWarps][TB][32];
-    const int h = blockIdx.y, c0 = blockIdx.x * 32, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int col = c0 + lane;
-    unsigned long long S[DR / 2];        // two neighbouring state rows each
-    float* sbase = state + ((size_t)h * d + warp * DR) * dv + col;
+// Sum of v[i] over the warp's lanes, for 32 values at once: lane i gets the total of v[i].
+__device__ __forceinline__ float transpose_sum(float (&v)[32], int lane) {
 #pragma unroll
-    for (int r = 0; r < DR; r += 2) {
-        const int i = warp * DR + r;
-        S[r / 2] = pack2(i < d && col < dv ? sbase[(size_t)r * dv] : 0.f, i + 1 < d && col < dv ? sbase[(size_t)(r + 1) * dv] : 0.f);
-    }
-    float pg[PER], pq[PER], pv[PERV];
-    auto fetch = [&](int t0) {
+    for (int s = 16; s > 0; s >>= 1)
 #pragma unroll
-        for (int i = 0; i < PER; i++) {
-            const int e = tid + i * kWarps * 32, t = e / D, c = e % D;
-            const bool in = t0 + t < M && c < d;
-            pg[i] = in ? gf[((size_t)(t0 + t) * H + h) * d + c] : 0.f;
-            pq[i] = in ? to_f32<T>(q[((size_t)(t0 + t) * H + h) * d + c]) : 0.f;
+        for (int i = 0; i < s; i++) {
+            const bool up = (lane & s) != 0;
+            const float keep = up ? v[i + s] : v[i], send = up ? v[i] : v[i + s];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, send, s);
         }
+    return v[0];
+}
+
+// RPL neighbouring values of a shared-memory row as packed pairs.
+template <int RPL> __device__ __forceinline__ void ld_pairs(unsigned long long (&r)[RPL / 2], const float* p) {
 #pragma unroll
-        for (int i = 0; i < PERV; i++) {
-            const int e = tid + i * kWarps * 32, t = e / 32, c = c0 + (e & 31);
-            pv[i] = (t < TB && t0 + t < M && c < dv) ? to_f32<T>(v[((size_t)(t0 + t) * H + h) * dv + c]) : 0.f;
-        }
-    };
-    fetch(0);
-    for (int t0 = 0; t0 < M; t0 += TB) {
-        __syncthreads();                               // the previous block's parts have been read
+    for (int i = 0; i < RPL / 2; i++) r[i] = *reinterpret_cast<const unsigned long long*>(p + 2 * i);
+}
+template <int RPL> __device__ __forceinline__ void ld_pairs(unsigned long long (&r)[RPL / 2], const bf16* p) {
 #pragma unroll
-        for (int i = 0; i < PER; i++) {
-            const int e = tid + i * kWarps * 32;
-            (&sg[0][0])[e] = pg[i];
-            (&sq[0][0])[e] = pq[i];
-        }
-#pragma unroll
-        for (int i = 0; i < PERV; i++) {
-            const int e = tid + i * kWarps * 32;
-            if (e < TB * 32) (&sv[0][0])[e] = pv[i];
-        }
-        __syncthreads();
-        if (t0 + TB < M) fetch(t0 + TB);
-        const int nt = min(TB, M - t0);
-        auto token = [&](int t) {
-            const float vt = sv[t][lane];
-            const unsigned long long v2 = pack2(vt, vt);
-            unsigned long long a0 = 0ull, a1 = 0ull;
-#pragma unroll
-            for (int r = 0; r < DR; r += 4) {
-                const ulonglong2 g4 = *reinterpret_cast<const ulonglong2*>(&sg[t][warp * DR + r]);
-                const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(&sq[t][warp * DR + r]);
-                S[r / 2] = fma2(g4.x, fma2(S[r / 2], kMinusOne2, v2), S[r / 2]);
-                S[r / 2 + 1] = fma2(g4.y, fma2(S[r / 2 + 1], kMinusOne2, v2), S[r / 2 + 1]);
-                a0 = fma2(q4.x, S[r / 2], a0);
-                a1 = fma2(q4.y, S[r / 2 + 1], a1);
-            }
-            const float2 x = unpack2(a0), y = unpack2(a1);
-            part[warp][t][lane] = (x.x + x.y) + (y.x + y.y);
-        };
-        if (nt == TB) {
-#pragma unroll 4
-            for (int t = 0; t < TB; t++) token(t);
-        } else {
-            for (int t = 0; t < nt; t++) token(t);
-        }
-        __syncthreads();
-        for (int e = tid; e < nt * 32; e += kWarps * 32) {
-            const int t = e >> 5, c = e & 31;
-            float a = 0.f;
-#pragma unroll
-            for (int w = 0; w < kWarps; w++) a += part[w][t][c];
-            if (c0 + c < dv) o[((size_t)(t0 + t) * H + h) * dv + c0 + c] = a;
-        }
-    }
-#pragma unroll
-    for (int r = 0; r < DR; r += 2) {
-        const int i = warp * DR + r;
-        const float2 x = unpack2(S[r / 2]);
-        if (i < d && col < dv) sbase[(size_t)r * dv] = x.x;
-        if (i + 1 < d && col < dv) sbase[(size_t)(r + 1) * dv] = x.y;
+    for (int i = 0; i < RPL / 2; i++) {
+        const uint32_t u = *reinterpret_cast<const uint32_t*>(p + 2 * i);
+        r[i] = pack2(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u));
     }
 }
 
+// One row of `n` elements to shared memory by a warp: 16-byte asynchronous copies where the row allows them.
+template <typename E>
+__device__ __forceinline__ void fetch_row(E* dst, const E* src, int n, bool wide, int lane) {
+    constexpr int VE = 16 / (int)sizeof(E);
+    if (wide)
+        for (int c = lane * VE; c < n; c += 32 * VE) cp_async16(smem_u32(dst + c), src + c);
+    else
+        for (int c = lane; c < n; c += 32) dst[c] = src[c];
+}
+
+template <typename T, int RPL>           // state rows of a lane
+__global__ void __launch_bounds__(kWarps * 32) scan_kernel(const T* q, const float* gf, const T* v, float* state, float* o, int M, int H,
+                                                           int d, int dv) {
+    pdl_launch_dependents();
+    constexpr int D = 32 * RPL, TB = RPL == 8 ? 8 : 16, STAGES = 2;
+    __shared__ __align__(16) float sg[STAGES][TB][D];
+    __shared__ __align__(16) T sq[STAGES][TB][D];
+    __shared__ __align__(16) T sv[STAGES][TB][32];
+    const int h = blockIdx.y, c0 = blockIdx.x * 32, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int col = c0 + warp * kLaneCols, ncol = min(32, dv - c0);
+    const bool wide_g = d % 4 == 0, wide_q = d * (int)sizeof(T) % 16 == 0, wide_v = dv * (int)sizeof(T) % 16 == 0;
+    // what the copies never write stays zero: rows past the head's width, columns past its values
+    for (int i = tid; i < STAGES * TB; i += kWarps * 32) {
+        for (int c = d; c < D; c++) { sg[i / TB][i % TB][c] = 0.f; sq[i / TB][i % TB][c] = from_f32<T>(0.f); }
+        for (int c = ncol; c < 32; c++) sv[i / TB][i % TB][c] = from_f32<T>(0.f);
+    }
+    pdl_wait();
+    auto fetch = [&](int b) {
+        const int st = b % STAGES, t0 = b * TB;
+        for (int t = warp; t < TB && t0 + t < M; t += kWarps) {
+            const size_t row = (size_t)(t0 + t) * H + h;
+            fetch_row(sg[st][t], gf + row * d, d, wide_g, lane);
+            fetch_row(sq[st][t], q + row * d, d, wide_q, lane);
+            fetch_row(sv[st][t], v + row * dv + c0, ncol, wide_v, lane);
+        }
+        asm volatile("cp.async.commit_group;\n" ::: "memory");
+    };
+    fetch(0);
+    unsigned long long S[RPL / 2][kLaneCols];            // two neighbouring state rows each
+    float* sbase = state + ((size_t)h * d + lane * RPL) * dv + col;
+#pragma unroll
+    for (int r = 0; r < RPL; r += 2)
+#pragma unroll
+        for (int c = 0; c < kLaneCols; c++) {
+            const int i = lane * RPL + r;
+            S[r / 2][c] = pack2(i < d && col + c < dv ? sbase[(size_t)r * dv + c] : 0.f,
+                                i + 1 < d && col + c < dv ? sbase[(size_t)(r + 1) * dv + c] : 0.f);
+        }
+    const int nb = (M + TB - 1) / TB;
+    for (int b = 0; b < nb; b++) {
+        const int st = b % STAGES, t0 = b * TB;
+        asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+        __syncthreads();                                 // this block is here, the one before has been read
+        if (b + 1 < nb) fetch(b + 1);
+#pragma unroll 1
+        for (int tg = 0; tg < TB && t0 + tg < M; tg += 8) {
+            const int nt = min(8, M - t0 - tg);
+            float y[32];                                 // [token][column], this lane's rows
+#pragma unroll
+            for (int t = 0; t < 8; t++) {
+                if (t < nt) {
+                    unsigned long long g2[RPL / 2], q2[RPL / 2], acc[kLaneCols], v2[kLaneCols];
+                    ld_pairs<RPL>(g2, &sg[st][tg + t][lane * RPL]);
+                    ld_pairs<RPL>(q2, &sq[st][tg + t][lane * RPL]);
+#pragma unroll
+                    for (int c = 0; c < kLaneCols; c++) {
+                        const float x = to_f32<T>(sv[st][tg + t][warp * kLaneCols + c]);
+                        v2[c] = pack2(x, x);
+                        acc[c] = 0ull;
+                    }
+#pragma unroll
+                    for (int r = 0; r < RPL / 2; r++) {
+#pragma unroll
+                        for (int c = 0; c < kLaneCols; c++) {
+                            S[r][c] = fma2(g2[r], fma2(S[r][c], kMinusOne2, v2[c]), S[r][c]);
+                            acc[c] = fma2(q2[r], S[r][c], acc[c]);
+                        }
+                    }
+#pragma unroll
+                    for (int c = 0; c < kLaneCols; c++) {
+                        const float2 x = unpack2(acc[c]);
+                        y[t * kLaneCols + c] = x.x + x.y;
+                    }
+                } else {
+#pragma unroll
+                    for (int c = 0; c < kLaneCols; c++) y[t * kLaneCols + c] = 0.f;
+                }
+            }
+            const float out = transpose_sum(y, lane);
+            const int t = lane / kLaneCols, c = col + lane % kLaneCols;
+            if (t < nt && c < dv) o[((size_t)(t0 + tg + t) * H + h) * dv + c] = out;
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < RPL; r += 2)
+#pragma unroll
+        for (int c = 0; c < kLaneCols; c++) {
+            const int i = lane * RPL + r;
+            const float2 x = unpack2(S[r / 2][c]);
+            if (i < d && col + c < dv) sbase[(size_t)r * dv + c] = x.x;
+            if (i + 1 < d && col + c < dv) sbase[(size_t)(r + 1) * dv + c] = x.y;
+        }
+}
+
 template <typename T>
-__global__ void __launch_bounds__(128) tree_kernel(const T* __restrict__ q, const float* __restrict__ pend_g, const T* __restrict__ pend_v,
-                                                   const float* __restrict__ state, const unsigned long long* __restrict__ mask,
-                                                   float* __restrict__ o, int H, int d, int dv) {
+__global__ void __launch_bounds__(128) tree_kernel(const T* q, const float* pend_g, const T* pend_v,
+                                                   const float* state, const unsigned long long* mask,
+                                                   float* o, int H, int d, int dv) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float sw[B200_HYBRID_PENDING][4];
@@ -179,7 +220,7 @@ __global__ void __launch_bounds__(128) tree_kernel(const T* __restrict__ q, cons
 }
 
 template <typename T>
-__global__ void __launch_bounds__(128) head_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, T* __restrict__ out, int M, int H,
+__global__ void __launch_bounds__(128) head_norm_kernel(const float* o, const float* w, T* out, int M, int H,
                                                         int dv, int pitch, float eps) {
     pdl_launch_dependents();
     pdl_wait();
@@ -274,10 +315,10 @@ int launch_scan(const b200_hybrid_model& m, const b200_hybrid_layer& l, float* s
     const dim3 grid((l.vdim + 31) / 32, l.heads), block(kWarps * 32);
     const T* q = static_cast<const T*>(m.qb);
     const T* v = static_cast<const T*>(m.vb);
-    if (l.dim <= 32) launch_kernel(scan_kernel<T, 4, 16>, grid, block, 0, st, q, m.gf, v, state, m.o32, M, l.heads, l.dim, l.vdim);
-    else if (l.dim <= 64) launch_kernel(scan_kernel<T, 8, 16>, grid, block, 0, st, q, m.gf, v, state, m.o32, M, l.heads, l.dim, l.vdim);
-    else if (l.dim <= 128) launch_kernel(scan_kernel<T, 16, 16>, grid, block, 0, st, q, m.gf, v, state, m.o32, M, l.heads, l.dim, l.vdim);
-    else launch_kernel(scan_kernel<T, 32, 8>, grid, block, 0, st, q, m.gf, v, state, m.o32, M, l.heads, l.dim, l.vdim);
+    const float* gf = m.gf;
+    if (l.dim <= 64) launch_kernel(scan_kernel<T, 2>, grid, block, 0, st, q, gf, v, state, m.o32, M, l.heads, l.dim, l.vdim);
+    else if (l.dim <= 128) launch_kernel(scan_kernel<T, 4>, grid, block, 0, st, q, gf, v, state, m.o32, M, l.heads, l.dim, l.vdim);
+    else launch_kernel(scan_kernel<T, 8>, grid, block, 0, st, q, gf, v, state, m.o32, M, l.heads, l.dim, l.vdim);
     return check_launch();
 }
 

@@ -8,9 +8,9 @@ namespace {
 
 // ---- embedding: h[m,:] = dequant(E[tokens[m], :]) --------------------------------------------
 // One thread per uint32 pack (8 weights).  Same dequantisation as the matmul (q*s+b rounded once).
-__global__ void embed_gather_kernel(const int* __restrict__ tokens, const uint32_t* __restrict__ wq,
-                                    const __half* __restrict__ scales, const __half* __restrict__ biases,
-                                    __half* __restrict__ out, int M, int H, int V) {
+__global__ void embed_gather_kernel(const int* tokens, const uint32_t* wq,
+                                    const __half* scales, const __half* biases,
+                                    __half* out, int M, int H, int V) {
     pdl_wait();
     pdl_launch_dependents();
     const int m = blockIdx.y;
@@ -30,8 +30,8 @@ __global__ void embed_gather_kernel(const int* __restrict__ tokens, const uint32
 
 // ---- RMSNorm: y = fp16( (x * rsqrt(mean(x^2) + eps)) * w ), fp32 math --------------------------
 // One CTA per output row; `row_index` (optional, device) selects the source row of output row 0.
-__global__ void rms_norm_kernel(const __half* __restrict__ x, const __half* __restrict__ w,
-                                __half* __restrict__ y, const int* __restrict__ row_index, int H, float eps) {
+__global__ void rms_norm_kernel(const __half* x, const __half* w,
+                                __half* y, const int* row_index, int H, float eps) {
     pdl_wait();
     pdl_launch_dependents();
     __shared__ float red[32];
@@ -69,10 +69,10 @@ __global__ void rms_norm_kernel(const __half* __restrict__ x, const __half* __re
 // q is rotated in place; k is rotated and stored, v stored, at cache row  prefix + write_off + m.
 // Rotation (non-traditional / half-split layout), fp32 math:
 //   theta = (scaling * inv_freq[i]) * pos ;  (x[i], x[i+hd/2]) -> (x1 cos - x2 sin, x1 sin + x2 cos)
-__global__ void rope_kv_append_kernel(__half* __restrict__ qkv, const int* __restrict__ pos,
-                                      const float* __restrict__ inv_freq, float scaling,
-                                      __half* __restrict__ kcache, __half* __restrict__ vcache,
-                                      const int* __restrict__ prefix, int write_off, int Hq, int Hkv,
+__global__ void rope_kv_append_kernel(__half* qkv, const int* pos,
+                                      const float* inv_freq, float scaling,
+                                      __half* kcache, __half* vcache,
+                                      const int* prefix, int write_off, int Hq, int Hkv,
                                       int hd, int cap) {
     pdl_wait();
     pdl_launch_dependents();
@@ -109,7 +109,7 @@ __global__ void rope_kv_append_kernel(__half* __restrict__ qkv, const int* __res
 
 // ---- tensor-parallel epilogue: h = fp16(h + fp16(sum)) where `sum` holds the all-reduced fp32 partial
 // products of a row-parallel linear layer (the rounding points of the unsharded residual epilogue).
-__global__ void residual_add_f32_kernel(__half* __restrict__ h, const float* __restrict__ sum, int n) {
+__global__ void residual_add_f32_kernel(__half* h, const float* sum, int n) {
     pdl_wait();
     pdl_launch_dependents();
     const int i = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
@@ -122,7 +122,7 @@ __global__ void residual_add_f32_kernel(__half* __restrict__ h, const float* __r
 
 // ---- element-wise halves of the fused matmul epilogues, for prompt ingestion through the large-M matmul (whose own
 // epilogue is plain): the same rounding points as B200_EPI_RESIDUAL and B200_EPI_SILU_MUL.
-__global__ void add_f16_kernel(__half* __restrict__ h, const __half* __restrict__ y, size_t n) {
+__global__ void add_f16_kernel(__half* h, const __half* y, size_t n) {
     pdl_wait();
     pdl_launch_dependents();
     const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 8;
@@ -136,7 +136,7 @@ __global__ void add_f16_kernel(__half* __restrict__ h, const __half* __restrict_
     *reinterpret_cast<uint4*>(h + i) = a;
 }
 
-__global__ void silu_mul_f16_kernel(const __half* __restrict__ gate, const __half* __restrict__ up, __half* __restrict__ out,
+__global__ void silu_mul_f16_kernel(const __half* gate, const __half* up, __half* out,
                                     size_t n) {
     pdl_wait();
     pdl_launch_dependents();
@@ -157,9 +157,9 @@ __global__ void silu_mul_f16_kernel(const __half* __restrict__ gate, const __hal
 }
 
 // Stand-alone operator with the reference's tensor layout: in/out (B, H, L, D), offsets (B, L).
-__global__ void rope_positions_kernel(const __half* __restrict__ in, const int* __restrict__ offsets,
-                                      const float* __restrict__ inv_freq, float scaling,
-                                      __half* __restrict__ out, int H, int Lq, int D) {
+__global__ void rope_positions_kernel(const __half* in, const int* offsets,
+                                      const float* inv_freq, float scaling,
+                                      __half* out, int H, int Lq, int D) {
     pdl_wait();
     pdl_launch_dependents();
     const int l = blockIdx.x, h = blockIdx.y, b = blockIdx.z;

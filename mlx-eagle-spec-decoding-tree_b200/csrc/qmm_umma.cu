@@ -84,7 +84,7 @@ __device__ __forceinline__ bool uwait(uint32_t bar, uint32_t parity) {
     return mbar_wait_timed(bar, parity, kUmmaWaitPolls, 32u);
 }
 
-__global__ void x_canonical_kernel(const __half* __restrict__ x, __half* __restrict__ xc, int M, int K, int NT) {
+__global__ void x_canonical_kernel(const __half* x, __half* xc, int M, int K, int NT) {
     pdl_wait();
     pdl_launch_dependents();
     // one 16-byte unit (token, k group of 8) per thread

@@ -102,7 +102,7 @@ __device__ __forceinline__ float score_of(float logit, double lse) {
 }
 
 // ---------------------------------------------------------------- row kernels over logits [R, V]
-__global__ void row_max_kernel(const __half* __restrict__ logits, int V, uint32_t* __restrict__ row_max) {
+__global__ void row_max_kernel(const __half* logits, int V, uint32_t* row_max) {
     pdl_wait();
     pdl_launch_dependents();
     const int r = blockIdx.y;
@@ -117,8 +117,8 @@ __global__ void row_max_kernel(const __half* __restrict__ logits, int V, uint32_
 
 // temp: temperature the logits are divided by before the exponential (1.0: the plain soft-max; dividing by 1.0 is exact,
 // so the draft tree's log-probabilities are what they were).
-__global__ void row_sumexp_kernel(const __half* __restrict__ logits, int V, const uint32_t* __restrict__ row_max,
-                                  unsigned long long* __restrict__ row_sum, double temp) {
+__global__ void row_sumexp_kernel(const __half* logits, int V, const uint32_t* row_max,
+                                  unsigned long long* row_sum, double temp) {
     pdl_wait();
     pdl_launch_dependents();
     const int r = blockIdx.y;
@@ -135,10 +135,10 @@ __global__ void row_sumexp_kernel(const __half* __restrict__ logits, int V, cons
 
 // Local top-8 of one chunk of one row.  by_score == 0: order by the raw logit (root expansion,
 // mlx_eagle.py:411); by_score == 1: order by the fp32 log-probability (tree levels, :104-105).
-__global__ void __launch_bounds__(256) row_topk_kernel(const __half* __restrict__ logits, int V,
-                                                       const uint32_t* __restrict__ row_max,
-                                                       const unsigned long long* __restrict__ row_sum,
-                                                       int by_score, unsigned long long* __restrict__ cand) {
+__global__ void __launch_bounds__(256) row_topk_kernel(const __half* logits, int V,
+                                                       const uint32_t* row_max,
+                                                       const unsigned long long* row_sum,
+                                                       int by_score, unsigned long long* cand) {
     pdl_wait();
     pdl_launch_dependents();
     // Every thread keeps its 16 keys in registers; each warp selects the top 8 of its 512 keys with warp
@@ -191,7 +191,7 @@ __device__ __forceinline__ float logit_f32(__half v) { return __half2float(v); }
 __device__ __forceinline__ float logit_f32(float v) { return v; }
 
 template <typename L>
-__global__ void row_argmax_kernel(const L* __restrict__ logits, int V, unsigned long long* __restrict__ best_key) {
+__global__ void row_argmax_kernel(const L* logits, int V, unsigned long long* best_key) {
     pdl_wait();
     pdl_launch_dependents();
     const int r = blockIdx.y;
@@ -206,7 +206,7 @@ __global__ void row_argmax_kernel(const L* __restrict__ logits, int V, unsigned 
     if ((threadIdx.x & 31) == 0) atomicMax(best_key + r, best);
 }
 
-__global__ void argmax_key_shift_kernel(unsigned long long* __restrict__ best_key, int R, unsigned int index_offset) {
+__global__ void argmax_key_shift_kernel(unsigned long long* best_key, int R, unsigned int index_offset) {
     pdl_wait();
     pdl_launch_dependents();
     const int r = threadIdx.x;
@@ -342,7 +342,7 @@ __global__ void __launch_bounds__(256) tree_expand_kernel(const ExpandParams p) 
 // ---------------------------------------------------------------- catch-up pass inputs
 // The draft model re-reads the tokens accepted in the previous step plus the bonus token, padded
 // with zeros to 8 rows (mlx_eagle.py:400-408); logits of row `accept_len` are the ones used.
-__global__ void prep_catchup_kernel(const int* __restrict__ ctl, const int* __restrict__ y, int* fwd_tokens,
+__global__ void prep_catchup_kernel(const int* ctl, const int* y, int* fwd_tokens,
                                     int* fwd_pos, unsigned long long* fwd_mask, int* fwd_prefix, int* sel_row) {
     pdl_wait();
     pdl_launch_dependents();
@@ -565,7 +565,7 @@ __global__ void tree_accept_kernel(const AcceptParams p) {
 }
 
 // ---------------------------------------------------------------- decoding without a draft (a tree of the root alone)
-__global__ void prep_root_kernel(const int* __restrict__ ctl, const int* __restrict__ y, int* fwd_tokens, int* fwd_pos,
+__global__ void prep_root_kernel(const int* ctl, const int* y, int* fwd_tokens, int* fwd_pos,
                                  unsigned long long* fwd_mask, int* fwd_prefix) {
     pdl_wait();
     pdl_launch_dependents();
@@ -778,9 +778,9 @@ __global__ void __launch_bounds__(256) bonus_pick_kernel(const SampleParams p) {
 // ---------------------------------------------------------------- KV compaction of the accepted path
 // For every layer and kv head: rows old_base+1 .. old_base+a  <-  rows old_base + node[j]
 // (mlx_eagle.py:366-374).  Sources are gathered before any store (array-assignment semantics).
-__global__ void kv_compact_kernel(__half* __restrict__ cache, size_t layer_stride, size_t kv_stride,
-                                  int cap, int hd, const int* __restrict__ accept_rows,
-                                  const int* __restrict__ ctl) {
+__global__ void kv_compact_kernel(__half* cache, size_t layer_stride, size_t kv_stride,
+                                  int cap, int hd, const int* accept_rows,
+                                  const int* ctl) {
     pdl_wait();
     pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char smem_raw[];
