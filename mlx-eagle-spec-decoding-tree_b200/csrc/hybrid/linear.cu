@@ -338,14 +338,9 @@ int launch_gemm(const b200_linear& lin, const void* x, int x_rows, const Epi& ep
     p.ksplit = 1;
     const int sms = sm_count(), tiles = p.ntiles * p.ttiles;
     if (NT <= 128) {
-        // Cut K so that the tiles' slices cover the SMs evenly: one CTA per SM where that uses most of them (its neighbour
-        // in the stream can then sit beside it and fetch weights ahead), else two.
-        float best = 0.f;
-        for (int k = 1; k <= kMaxSplit && k * 2 <= p.kblocks && tiles * k <= sms * G::PER_SM; k++) {
-            const int per_sm = (tiles * k + sms - 1) / sms;
-            const float used = (float)(tiles * k) / (float)(sms * per_sm) - (per_sm > 1 ? 0.1f : 0.f);
-            if (used > best) { best = used; p.ksplit = k; }
-        }
+        // Cut K while the slices of all tiles fit the device at once (two CTAs per SM keep enough copies in flight) and are
+        // at least two blocks long.  Powers of two: clusters of other sizes do not fill the SM groups.
+        while (p.ksplit < kMaxSplit && tiles * p.ksplit * 2 <= sms * G::PER_SM && p.kblocks >= 4 * p.ksplit) p.ksplit *= 2;
     }
     int grid = tiles * p.ksplit;
     if (p.ksplit == 1 && G::NACC > 1 && grid > sms) grid = sms;     // persistent

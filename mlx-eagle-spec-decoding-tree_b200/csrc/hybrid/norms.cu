@@ -36,16 +36,23 @@ template <int V> __device__ __forceinline__ void st(bf16* p, const Vec<V>& r) {
     }
 }
 
-__global__ void __launch_bounds__(kThreads) embed_kernel(const int* tokens, const bf16* table, int width, int vocab,
-                                                         float* x, float* emb) {
+__global__ void __launch_bounds__(kThreads) embed_kernel(const int* tokens, const bf16* table, int width, int vocab, float* x, float* emb) {
     pdl_launch_dependents();
     pdl_wait();
-    const int m = blockIdx.x;
+    constexpr int N = 4;                              // channels of a thread; all loads before the first store
+    const int m = blockIdx.x, c0 = blockIdx.y * kThreads * N + threadIdx.x;
     const int tok = min(max(tokens[m], 0), vocab - 1);
-    for (int c = threadIdx.x; c < width; c += kThreads) {
-        const float v = __bfloat162float(table[(size_t)tok * width + c]);
-        x[(size_t)m * width + c] = v;
-        if (emb != nullptr) emb[(size_t)m * width + c] = v;
+    const bf16* src = table + (size_t)tok * width;
+    bf16 v[N];
+#pragma unroll
+    for (int i = 0; i < N; i++) v[i] = c0 + i * kThreads < width ? src[c0 + i * kThreads] : __float2bfloat16_rn(0.f);
+#pragma unroll
+    for (int i = 0; i < N; i++) {
+        const int c = c0 + i * kThreads;
+        if (c < width) {
+            x[(size_t)m * width + c] = __bfloat162float(v[i]);
+            if (emb != nullptr) emb[(size_t)m * width + c] = __bfloat162float(v[i]);
+        }
     }
 }
 
@@ -242,7 +249,7 @@ __global__ void add_kernel(float* x, const float* y, size_t n) {
 }  // namespace
 
 int launch_embed(const b200_hybrid_model& m, const b200_hybrid_pass& p, cudaStream_t st) {
-    launch_kernel(embed_kernel, dim3(p.M), dim3(kThreads), 0, st, p.tokens, static_cast<const bf16*>(m.embed), m.width, m.vocab, m.x,
+    launch_kernel(embed_kernel, dim3(p.M, (m.width + 4 * kThreads - 1) / (4 * kThreads)), dim3(kThreads), 0, st, p.tokens, static_cast<const bf16*>(m.embed), m.width, m.vocab, m.x,
                   m.injects ? m.emb : static_cast<float*>(nullptr));
     return check_launch();
 }

@@ -105,14 +105,23 @@ __global__ void __launch_bounds__(kWarps * 32) scan_kernel(const T* q, const flo
     fetch(0);
     unsigned long long S[RPL / 2][kLaneCols];            // two neighbouring state rows each
     float* sbase = state + ((size_t)h * d + lane * RPL) * dv + col;
+    const bool wide_s = dv % 4 == 0 && col < dv;
+    float row[RPL][kLaneCols];
+#pragma unroll
+    for (int r = 0; r < RPL; r++) {
+        const bool in = lane * RPL + r < d;
+        if (wide_s) {
+            const float4 x = in ? *reinterpret_cast<const float4*>(sbase + (size_t)r * dv) : make_float4(0.f, 0.f, 0.f, 0.f);
+            row[r][0] = x.x; row[r][1] = x.y; row[r][2] = x.z; row[r][3] = x.w;
+        } else {
+#pragma unroll
+            for (int c = 0; c < kLaneCols; c++) row[r][c] = in && col + c < dv ? sbase[(size_t)r * dv + c] : 0.f;
+        }
+    }
 #pragma unroll
     for (int r = 0; r < RPL; r += 2)
 #pragma unroll
-        for (int c = 0; c < kLaneCols; c++) {
-            const int i = lane * RPL + r;
-            S[r / 2][c] = pack2(i < d && col + c < dv ? sbase[(size_t)r * dv + c] : 0.f,
-                                i + 1 < d && col + c < dv ? sbase[(size_t)(r + 1) * dv + c] : 0.f);
-        }
+        for (int c = 0; c < kLaneCols; c++) S[r / 2][c] = pack2(row[r][c], row[r + 1][c]);
     const int nb = (M + TB - 1) / TB;
     for (int b = 0; b < nb; b++) {
         const int st = b % STAGES, t0 = b * TB;
@@ -159,14 +168,22 @@ __global__ void __launch_bounds__(kWarps * 32) scan_kernel(const T* q, const flo
         }
     }
 #pragma unroll
-    for (int r = 0; r < RPL; r += 2)
+    for (int r = 0; r < RPL; r++) {
+        if (lane * RPL + r >= d) break;
+        float x[kLaneCols];
 #pragma unroll
         for (int c = 0; c < kLaneCols; c++) {
-            const int i = lane * RPL + r;
-            const float2 x = unpack2(S[r / 2][c]);
-            if (i < d && col + c < dv) sbase[(size_t)r * dv + c] = x.x;
-            if (i + 1 < d && col + c < dv) sbase[(size_t)(r + 1) * dv + c] = x.y;
+            const float2 y = unpack2(S[r / 2][c]);
+            x[c] = r & 1 ? y.y : y.x;
         }
+        if (wide_s) {
+            *reinterpret_cast<float4*>(sbase + (size_t)r * dv) = make_float4(x[0], x[1], x[2], x[3]);
+        } else {
+#pragma unroll
+            for (int c = 0; c < kLaneCols; c++)
+                if (col + c < dv) sbase[(size_t)r * dv + c] = x[c];
+        }
+    }
 }
 
 template <typename T>
