@@ -23,7 +23,7 @@ length 0 and above: random-init pairs accept nothing, so the headline counts one
 Other workloads: ``c2`` draft-only tree build (0.5B-shape draft, prompt 128, depth 3, 7 nodes), ``c4``
 Llama-3-8B-shape target + Llama-3.2-1B-shape draft (prompt 1024, depth 4, 31 verify tokens, also reports the
 time to the first token of the 1024-token prompt), ``tp70b`` / ``tp7b`` one stream with the target cut across
-all ranks.  ``--impl reference`` times the CPU restatement only (the reference itself is MLX/Metal and cannot
+all ranks, ``hybrid`` the layer-list design beside the 4-bit models of equal size (plain decoding, prompts).  ``--impl reference`` times the CPU restatement only (the reference itself is MLX/Metal and cannot
 run on Linux), on the same configuration, and prints the same line with ``"impl": "reference"``.
 """
 from __future__ import annotations
