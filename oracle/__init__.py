@@ -21,4 +21,5 @@ qmm_ref     4-bit affine dequantise + matmul  (``kernels/progression/simd_no_swi
 detmath     deterministic exp/log used for log-probabilities
 tree_ref    tree build / finalise / accept / compaction  (``mlx_eagle.py``)
 model_ref   Llama/Qwen2 forward with tree hooks  (``mlx_llama.py``)
+hybrid_ref  layer-list decoders, one function per mechanism (no counterpart in the reference)
 """
