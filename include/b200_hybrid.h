@@ -25,14 +25,24 @@ extern "C" {
 
 #define B200_MIXER_ATTENTION 0  /* softmax attention, 1 or 2 maps per head (2: differential), window + kept first keys */
 #define B200_MIXER_RECURRENCE 1 /* gated linear recurrence, S += (1-f) (v - S) per channel row, o = S^T q              */
+#define B200_MIXER_DELTA 2      /* gated delta rule with a decay per key channel, convolutions on q, k, v              */
+#define B200_MIXER_LATENT 3     /* softmax attention over a shared low-rank latent and one rotated key part            */
+
+#define B200_FF_POLYNORM 0 /* W_down polynorm(W_up h)                                                                  */
+#define B200_FF_GATED 1    /* W_down (gelu_tanh(W_gate h + b) * (W_up h + b)) + b                                      */
+#define B200_FF_EXPERTS 2  /* sum over the chosen experts of W_down (swish_alpha(min(g, l)) * (clamp(u, l) + shift))   */
 
 #define B200_HYBRID_PENDING 64 /* rows of a request whose inputs are kept until they are committed */
 #define B200_HYBRID_MAX_TAPS 8
+#define B200_HYBRID_MAX_EXPERTS 512
+#define B200_HYBRID_MAX_TOP 16
 
-/* y = x W^T; W bf16 [n rounded up to 128][pitch], pitch = k rounded up to 64, rows past n and columns past k zero. */
+/* y = x W^T; W bf16 [n rounded up to 128][pitch], pitch = k rounded up to 64, rows past n and columns past k zero.
+ * groups > 1: a stack of such matrices, each over pitch columns of x of its own (group g reads x columns g*pitch.. and gives
+ * output columns g*n ..). */
 typedef struct b200_linear {
     const void* w;
-    int n, k, pitch, reserved;
+    int n, k, pitch, groups;
 } b200_linear;
 
 typedef struct b200_hybrid_layer {
@@ -42,16 +52,39 @@ typedef struct b200_hybrid_layer {
     int window, keep_first;             /* position i sees j <= i with i - j < window or j < keep_first              */
     int ff;                             /* feed-forward width, 0: the layer has none                                 */
     float scale, lambda, out_scale;     /* score scale; maps = 2: weight of map 2, factor after the head's norm      */
-    float act[4];                       /* a N(z) + b N(z^2) + c N(z^3) + e                                          */
-    int reserved;
+    float act[4];                       /* polynorm: a N(z) + b N(z^2) + c N(z^3) + e; experts: limit, alpha, shift  */
+    int ff_kind;
     const float* norm1;                 /* [width] multiplicative weights (1 + w already added where w is zero-centred) */
     const float* norm2;
     const float* conv;                  /* [taps][width]                                                             */
     const float* gate_bias;             /* recurrence: bias and lower bound of the forget gate [heads * dim]         */
     const float* gate_lower;
     const float* head_norm;             /* recurrence: [vdim]                                                        */
-    b200_linear in;                     /* rows q | k | v | gate (attention), q | f | v (recurrence)                 */
-    b200_linear out, up, down;
+    b200_linear in;                     /* rows q | k | v | gate (attention), q | f | v (recurrence),
+                                           q | k | v | beta | low-rank inputs (delta), unrotated queries | rotated query
+                                           parts | latent | rotated key part (latent)                                */
+    b200_linear out, up, down;          /* gated kinds: rows of `up` alternate gate, up; experts: groups = experts   */
+    /* delta */
+    int conv_taps;                      /* taps of the convolutions on q, k, v                                       */
+    int low_rank;                       /* columns of the low-rank inputs of decay and output gate together          */
+    const float* mix_conv;              /* [conv_taps][2*kv_heads*dim + heads*vdim], last tap: the current token     */
+    const float* decay_bias;            /* [heads*dim]                                                               */
+    const float* decay_rate;            /* [heads*dim]: g = exp(-rate * softplus(z + bias))                          */
+    b200_linear low;                    /* rows decay | output gate over the low-rank inputs                         */
+    /* latent */
+    int kv_rank, rot_dim;
+    float rot_mag;                      /* factor on cos and sin                                                     */
+    int reserved;
+    const float* rot_freq;              /* [rot_dim / 2] angle per position                                          */
+    const float* latent_norm;           /* [kv_rank]                                                                 */
+    b200_linear absorb;                 /* groups = heads: unrotated query -> its form over the latent               */
+    b200_linear value;                  /* groups = heads: latent -> value                                           */
+    b200_linear expand;                 /* rows unrotated keys | values of all heads over the latent                 */
+    /* gated feed-forwards and experts */
+    int experts, top;
+    const float* up_bias;               /* [2*ff], alternating like the rows of `up`                                 */
+    const float* down_bias;             /* [width]                                                                   */
+    b200_linear router;
 } b200_hybrid_layer;
 
 /* One execution of a layer in a pass (a repeated layer has one per repetition), with the place of its cache / state
@@ -60,9 +93,12 @@ typedef struct b200_hybrid_run {
     int layer;
     int inject;                         /* the embedding output is added to the residual stream after this run       */
     long long conv_off;                 /* fp32 [taps - 1][width], oldest first                                      */
-    long long k_off, v_off;             /* attention: [kv_heads][rows][maps * dim16], [kv_heads][rows][vdim16]       */
-    long long state_off;                /* recurrence: fp32 [heads][dim][vdim]                                       */
+    long long k_off, v_off;             /* attention: [kv_heads][rows][maps * dim16], [kv_heads][rows][vdim16];
+                                           latent: k_off [rows][kv_rank16 + rot_dim16]                               */
+    long long state_off;                /* recurrence: fp32 [heads][dim][vdim], delta: fp32 [heads][vdim][dim]       */
     long long pend_h, pend_g, pend_v;   /* fp32 [64][width], fp32 [64][heads*dim], activations [64][heads*vdim]      */
+    long long mix_off;                  /* delta: activations [conv_taps - 1][channels], oldest first                */
+    long long pend_c, pend_k, pend_b;   /* delta: activations [64][channels], fp32 [64][kv_heads*dim], fp32 [64][heads] */
 } b200_hybrid_run;
 
 typedef struct b200_hybrid_model {
@@ -70,7 +106,8 @@ typedef struct b200_hybrid_model {
     int injects;                        /* some run injects: the embedding output is kept during the pass            */
     int conv_max_taps;
     float eps, residual_mult, softcap;  /* softcap <= 0: none                                                        */
-    int reserved;
+    int norm_out;                       /* 0: sublayers read the normed stream; 1: they read the stream, their outputs are
+                                           normed before they are added (residual_mult unused)                       */
     const void* embed;                  /* bf16 [vocab][width]                                                       */
     const float* final_norm;
     const b200_hybrid_layer* layers;    /* HOST                                                                      */
@@ -89,7 +126,22 @@ typedef struct b200_hybrid_model {
     float* o32;                         /* recurrence output [max_rows][heads * vdim]                                */
     void* ab;                           /* mixer output [max_rows][heads * vdim rounded up to 64]                    */
     void* zb;                           /* feed-forward [max_rows][ff64], before and after the activation            */
-    void* zab;
+    void* zab;                          /* (experts: max_rows * top rows)                                            */
+    float* y;                           /* sublayer output before its norm / expert outputs [max_rows * top][width]  */
+    void* cb;                           /* delta: convolution inputs [max_rows][channels]                            */
+    void* lowb;                         /* delta: low-rank inputs [max_rows][low_rank64]                             */
+    float* q32;                         /* delta: unit queries and keys [max_rows][kv_heads*dim]                     */
+    float* k32;
+    float* beta;                        /* delta: [max_rows][heads]                                                  */
+    float* lat32;                       /* latent: rotated query parts | latent | rotated key part, before norm and rotation */
+    void* qn;                           /* latent: unrotated queries [max_rows][heads][dim64]                        */
+    void* ob;                           /* latent: attention output over the latent [max_rows][heads][kv_rank64]     */
+    void* kx;                           /* latent: keys and values of all heads for `x_rows` cache rows, prompts     */
+    void* vx;
+    float* zr;                          /* experts: router logits [max_rows][experts]                                */
+    int* route;                         /* experts: see b200_hybrid_route_ints                                       */
+    void* xg;                           /* experts: gathered inputs [max_rows * top][width64]                        */
+    int x_rows, route_top, route_experts, reserved;
     void* pending;
     float* attn_part;                   /* attention partials                                                        */
     size_t attn_part_bytes;
@@ -119,6 +171,9 @@ typedef struct b200_hybrid_pass {
 
 /* Bytes of attention partials a pass of `rows` tree rows (or fp32 / short chain rows) needs at most. */
 size_t b200_hybrid_attention_workspace_bytes(const b200_hybrid_model* model, int rows);
+
+/* Ints of `route`: expert and position of every (row, choice), the choices' scores, first place of every expert. */
+size_t b200_hybrid_route_ints(int max_rows, int top, int experts);
 
 int b200_hybrid_forward(const b200_hybrid_model* model, const b200_hybrid_pass* pass, void* stream);
 

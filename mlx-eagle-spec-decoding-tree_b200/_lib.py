@@ -59,6 +59,8 @@ def hybrid() -> ctypes.CDLL:
         l.b200_hybrid_set_pdl.argtypes = [i32]
         l.b200_hybrid_attention_workspace_bytes.restype = sz
         l.b200_hybrid_attention_workspace_bytes.argtypes = [mp, i32]
+        l.b200_hybrid_route_ints.restype = sz
+        l.b200_hybrid_route_ints.argtypes = [i32, i32, i32]
         l.b200_hybrid_forward.restype = i32
         l.b200_hybrid_forward.argtypes = [mp, pp, vp]
         l.b200_hybrid_commit.restype = i32
@@ -198,7 +200,7 @@ class ForwardDesc(ctypes.Structure):
 
 class Linear(ctypes.Structure):
     """Mirror of ``b200_linear`` (include/b200_hybrid.h)."""
-    _fields_ = [("w", ctypes.c_void_p)] + [(n, ctypes.c_int) for n in ("n", "k", "pitch", "reserved")]
+    _fields_ = [("w", ctypes.c_void_p)] + [(n, ctypes.c_int) for n in ("n", "k", "pitch", "groups")]
 
 
 class HybridLayer(ctypes.Structure):
@@ -206,27 +208,37 @@ class HybridLayer(ctypes.Structure):
     _fields_ = ([(n, ctypes.c_int) for n in ("mixer", "taps", "heads", "kv_heads", "dim", "vdim", "maps", "window",
                                              "keep_first", "ff")]
                 + [(n, ctypes.c_float) for n in ("scale", "lambda_", "out_scale")]
-                + [("act", ctypes.c_float * 4), ("reserved", ctypes.c_int)]
+                + [("act", ctypes.c_float * 4), ("ff_kind", ctypes.c_int)]
                 + [(n, ctypes.c_void_p) for n in ("norm1", "norm2", "conv", "gate_bias", "gate_lower", "head_norm")]
-                + [(n, Linear) for n in ("in_", "out", "up", "down")])
+                + [(n, Linear) for n in ("in_", "out", "up", "down")]
+                + [(n, ctypes.c_int) for n in ("conv_taps", "low_rank")]
+                + [(n, ctypes.c_void_p) for n in ("mix_conv", "decay_bias", "decay_rate")] + [("low", Linear)]
+                + [("kv_rank", ctypes.c_int), ("rot_dim", ctypes.c_int), ("rot_mag", ctypes.c_float), ("reserved", ctypes.c_int)]
+                + [(n, ctypes.c_void_p) for n in ("rot_freq", "latent_norm")] + [(n, Linear) for n in ("absorb", "value", "expand")]
+                + [("experts", ctypes.c_int), ("top", ctypes.c_int)]
+                + [(n, ctypes.c_void_p) for n in ("up_bias", "down_bias")] + [("router", Linear)])
 
 
 class HybridRun(ctypes.Structure):
     """Mirror of ``b200_hybrid_run``."""
     _fields_ = ([("layer", ctypes.c_int), ("inject", ctypes.c_int)]
-                + [(n, ctypes.c_longlong) for n in ("conv_off", "k_off", "v_off", "state_off", "pend_h", "pend_g", "pend_v")])
+                + [(n, ctypes.c_longlong) for n in ("conv_off", "k_off", "v_off", "state_off", "pend_h", "pend_g", "pend_v", "mix_off",
+                                                   "pend_c", "pend_k", "pend_b")])
 
 
 class HybridModelDesc(ctypes.Structure):
     """Mirror of ``b200_hybrid_model``."""
     _fields_ = ([(n, ctypes.c_int) for n in ("act_type", "width", "vocab", "n_layers", "n_runs", "max_rows", "injects",
                                              "conv_max_taps")]
-                + [(n, ctypes.c_float) for n in ("eps", "residual_mult", "softcap")] + [("reserved", ctypes.c_int)]
+                + [(n, ctypes.c_float) for n in ("eps", "residual_mult", "softcap")] + [("norm_out", ctypes.c_int)]
                 + [(n, ctypes.c_void_p) for n in ("embed", "final_norm")]
                 + [("layers", ctypes.POINTER(HybridLayer)), ("runs", ctypes.POINTER(HybridRun))]
                 + [(n, ctypes.c_void_p) for n in ("dev_layers", "dev_runs")] + [("head", Linear)]
                 + [(n, ctypes.c_void_p) for n in ("x", "emb", "hb", "qb", "gb", "vb", "gf", "o32", "ab", "zb", "zab",
-                                                  "pending", "attn_part")]
+                                                  "y", "cb", "lowb", "q32", "k32", "beta", "lat32", "qn", "ob", "kx", "vx",
+                                                  "zr", "route", "xg")]
+                + [(n, ctypes.c_int) for n in ("x_rows", "route_top", "route_experts", "reserved")]
+                + [(n, ctypes.c_void_p) for n in ("pending", "attn_part")]
                 + [("attn_part_bytes", ctypes.c_size_t), ("error", ctypes.c_void_p)])
 
 

@@ -11,6 +11,10 @@
 // attention_prompt: bf16, many query rows of one sequence.  CTA = (64 query rows, head), four warps of 16 rows,
 // mma.sync with the key/value blocks double-buffered by cp.async; both maps share the value block.  The softmax weights
 // enter the value product as a pair of bf16 terms (value + remainder), which keeps them at fp32-like precision.
+//
+// Latent attention (one low-rank latent and one rotated key part per token, shared by all heads) uses both: few rows walk the
+// latent itself, with queries brought into its space and the key row's first columns as values (SHARED); prompts walk keys
+// and values written out per head, the rotated part taken from the cache (LATENT).
 #include "hybrid.cuh"
 #include "../pipeline.cuh"
 
@@ -25,16 +29,17 @@ constexpr int kRowThreads = 128;
 
 struct AttnParams {
     const void* q;            // [M][q_pitch]: (head, map) vectors of dp elements
-    const void* kc;           // [G][cap][maps * dp]
+    const void* kc;           // [G][cap][maps * dp]; LATENT: [H][cap][dp - rp]
     const void* vc;           // [G][cap][vp]
-    const void* gate;         // [M][H * vdim]
-    void* out;                // [M][out_pitch]
+    const void* gate;         // [M][H * vdim], or null
+    const void* krot;         // LATENT: [..][krot_pitch] rotated key parts of rp columns
+    void* out;                // [M][out_pitch], heads out_head apart
     float* part;              // [M][H * maps][splits][vp + 2]
     const int* pos;
     const int* tail_pos;
     const unsigned long long* mask;
     const int* prefix;
-    int M, H, G, maps, dim, dp, vdim, vp, cap, window, keep, tree, tail, q_pitch, out_pitch;
+    int M, H, G, maps, dim, dp, vdim, vp, cap, window, keep, tree, tail, q_pitch, out_pitch, out_head, rp, krot_pitch;
     int splits, qgroups, hpg; // key splits; query-head groups of a kv head and heads in each
     float scale_log2, lambda, out_scale, eps;
 };
@@ -56,7 +61,7 @@ struct KeyWalk {
     __device__ __forceinline__ int row(int u) const { return u < ns ? u : (u < nc ? wstart + u - ns : prefix + u - nc); }
 };
 
-template <typename T, int QN, int CR>    // query vectors (at most), columns per thread
+template <typename T, int QN, int CR, bool SHARED>    // query vectors (at most), columns per thread, values are the keys' first columns
 __global__ void __launch_bounds__(kRowThreads) attention_rows_kernel(const AttnParams p) {
     pdl_launch_dependents();
     pdl_wait();
@@ -70,7 +75,8 @@ __global__ void __launch_bounds__(kRowThreads) attention_rows_kernel(const AttnP
     float* sr = sl + QN;                                                 // [2 QN] rescale factor of this block
     int* srow = reinterpret_cast<int*>(sr + 2 * QN);                     // [kKeys] cache row of the block's keys, -1: not visible
     T* sk = reinterpret_cast<T*>(srow + kKeys);                          // [kKeys][KP]
-    T* sv = sk + kKeys * KP;                                             // [kKeys][vp]
+    T* sv = SHARED ? sk : sk + kKeys * KP;                               // [kKeys][VP]
+    const int vload = SHARED ? 0 : p.vp, VP = SHARED ? KP : p.vp;
     const int split = blockIdx.x, g = blockIdx.y / p.qgroups, qg = blockIdx.y % p.qgroups, m = blockIdx.z;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int R = p.H / p.G;
@@ -111,9 +117,9 @@ __global__ void __launch_bounds__(kRowThreads) attention_rows_kernel(const AttnP
         __syncthreads();
         for (int k = warp; k < kKeys; k += kRowThreads / 32) {           // a warp per key row, 16 bytes per lane
             const int r = srow[k];
-            for (int c = lane; c * VE < KE + p.vp; c += 32) {
+            for (int c = lane; c * VE < KE + vload; c += 32) {
                 const bool key = c * VE < KE;
-                T* dst = key ? sk + k * KP + c * VE : sv + k * p.vp + (c * VE - KE);
+                T* dst = key ? sk + k * KP + c * VE : sv + k * VP + (c * VE - KE);
                 const T* src = key ? kbase + (size_t)r * KE + c * VE : vbase + (size_t)r * p.vp + (c * VE - KE);
                 if (r >= 0) cp_async16(smem_u32(dst), src);
                 else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
@@ -173,7 +179,7 @@ __global__ void __launch_bounds__(kRowThreads) attention_rows_kernel(const AttnP
                 for (int k = 0; k < kKeys; k += 4) {                     // rows that are not visible: weight 0, value 0
                     float v[4];
 #pragma unroll
-                    for (int e = 0; e < 4; e++) v[e] = to_f32<T>(sv[(k + e) * p.vp + col]);
+                    for (int e = 0; e < 4; e++) v[e] = to_f32<T>(sv[(k + e) * VP + col]);
 #pragma unroll
                     for (int i = 0; i < QN; i++)
                         if (i < nq) {
@@ -199,7 +205,7 @@ __global__ void __launch_bounds__(kRowThreads) attention_rows_kernel(const AttnP
 }
 
 // Adds the key splits of one (row, head) and finishes the head.
-template <typename T>
+template <typename T, int CR>
 __global__ void __launch_bounds__(kRowThreads) attention_merge_kernel(const AttnParams p) {
     pdl_launch_dependents();
     pdl_wait();
@@ -222,9 +228,9 @@ __global__ void __launch_bounds__(kRowThreads) attention_merge_kernel(const Attn
     }
     __syncthreads();
     float ss = 0.f;
-    float o[2];                          // vdim <= 256: at most two columns per thread
+    float o[CR];
 #pragma unroll
-    for (int c = 0; c < 2; c++) {
+    for (int c = 0; c < CR; c++) {
         const int col = tid + c * kRowThreads;
         o[c] = 0.f;
         if (col < p.vdim) {
@@ -243,11 +249,11 @@ __global__ void __launch_bounds__(kRowThreads) attention_merge_kernel(const Attn
     float f = 1.f;
     if (p.maps == 2) f = rsqrtf(block_sum(ss, red) / (float)p.vdim + p.eps) * p.out_scale;
 #pragma unroll
-    for (int c = 0; c < 2; c++) {
+    for (int c = 0; c < CR; c++) {
         const int col = tid + c * kRowThreads;
         if (col < p.vdim) {
-            const float gt = to_f32<T>(static_cast<const T*>(p.gate)[((size_t)m * p.H + h) * p.vdim + col]);
-            static_cast<T*>(p.out)[(size_t)m * p.out_pitch + (size_t)h * p.vdim + col] = from_f32<T>(o[c] * f * gt);
+            const float gt = p.gate != nullptr ? to_f32<T>(static_cast<const T*>(p.gate)[((size_t)m * p.H + h) * p.vdim + col]) : 1.f;
+            static_cast<T*>(p.out)[(size_t)m * p.out_pitch + (size_t)h * p.out_head + col] = from_f32<T>(o[c] * f * gt);
         }
     }
 }
@@ -272,7 +278,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
     return *reinterpret_cast<const uint32_t*>(&v);
 }
 
-template <int VT, int MAPS>              // 16-column value tiles, maps per head
+template <int VT, int MAPS, bool LATENT> // 16-column value tiles, maps per head
 __global__ void __launch_bounds__(128) attention_prompt_kernel(const AttnParams p) {
     pdl_launch_dependents();
     pdl_wait();
@@ -285,7 +291,8 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const AttnParams 
     const int h = blockIdx.x, r0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * kQRows, g = h / (p.H / p.G);   // longest rows first
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, t = lane & 3;
     const int base_pos = p.prefix[0], qpos0 = base_pos + r0, qlast = base_pos + min(p.M, r0 + kQRows) - 1;
-    const bf16* kbase = static_cast<const bf16*>(p.kc) + (size_t)g * p.cap * KE;
+    const int kown = LATENT ? KE - p.rp : KE;                            // key columns of the head's own
+    const bf16* kbase = static_cast<const bf16*>(p.kc) + (size_t)g * p.cap * kown;
     const bf16* vbase = static_cast<const bf16*>(p.vc) + (size_t)g * p.cap * p.vp;
 
     const int kv = KE / 8, vv = p.vp / 8;
@@ -310,7 +317,9 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const AttnParams 
         for (int e = tid; e < kKeys * kv; e += 128) {
             const int r = e / kv, c = e - r * kv;
             bf16* dst = sk + (st * kKeys + r) * KP + c * 8;
-            if (k0 + r <= qlast) cp_async16(smem_u32(dst), kbase + (size_t)(k0 + r) * KE + c * 8);
+            const bf16* src = kbase + (size_t)(k0 + r) * kown + c * 8;
+            if (LATENT && c * 8 >= kown) src = static_cast<const bf16*>(p.krot) + (size_t)(k0 + r) * p.krot_pitch + (c * 8 - kown);
+            if (k0 + r <= qlast) cp_async16(smem_u32(dst), src);
             else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
         }
         for (int e = tid; e < kKeys * vv; e += 128) {
@@ -459,15 +468,15 @@ __global__ void __launch_bounds__(128) attention_prompt_kernel(const AttnParams 
     for (int e = 0; e < 2; e++) {
         const int m = r0 + warp * 16 + gq + 8 * e;
         if (m >= p.M) continue;
-        const bf16* gr = static_cast<const bf16*>(p.gate) + ((size_t)m * p.H + h) * p.vdim;
-        bf16* orow = static_cast<bf16*>(p.out) + (size_t)m * p.out_pitch + (size_t)h * p.vdim;
+        const bf16* gr = p.gate != nullptr ? static_cast<const bf16*>(p.gate) + ((size_t)m * p.H + h) * p.vdim : nullptr;
+        bf16* orow = static_cast<bf16*>(p.out) + (size_t)m * p.out_pitch + (size_t)h * p.out_head;
         const float f = e ? f1 : f0;
 #pragma unroll
         for (int n = 0; n < VT * 2; n++)
 #pragma unroll
             for (int d = 0; d < 2; d++) {
                 const int col = n * 8 + 2 * t + d;
-                if (col < p.vdim) orow[col] = __float2bfloat16_rn(o[0][n][2 * e + d] * f * __bfloat162float(gr[col]));
+                if (col < p.vdim) orow[col] = __float2bfloat16_rn(o[0][n][2 * e + d] * f * (gr != nullptr ? __bfloat162float(gr[col]) : 1.f));
             }
     }
 }
@@ -484,23 +493,34 @@ void pick_groups(int R, int maps, int* hpg, int* qgroups) {
     *hpg = (R + *qgroups - 1) / *qgroups;
 }
 
+constexpr size_t kMaxSmem = 227 * 1024;
+
+size_t rows_smem(const AttnParams& p, int qn, int elem, bool shared) {
+    const int KP = p.maps * p.dp + 16 / elem;
+    return (size_t)(qn * p.dp + qn * (kKeys + 4) + 4 * qn + kKeys) * 4 + (size_t)kKeys * (KP + (shared ? 0 : p.vp)) * elem;
+}
+
+template <typename T, int QN, int CR, bool SHARED>
+int launch_rows_c(AttnParams& p, cudaStream_t st) {
+    const size_t smem = rows_smem(p, QN, sizeof(T), SHARED);
+    if (smem > kMaxSmem) return B200_ELIMIT;
+    auto k = attention_rows_kernel<T, QN, CR, SHARED>;
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return check_launch();
+    launch_kernel(k, dim3(p.splits, p.G * p.qgroups, p.M), dim3(kRowThreads), smem, st, p);
+    if (check_launch() != B200_OK) return B200_ECUDA;
+    launch_kernel(attention_merge_kernel<T, CR>, dim3(p.H, p.M), dim3(kRowThreads), 0, st, p);
+    return check_launch();
+}
+
 template <typename T, int QN>
 int launch_rows(AttnParams& p, cudaStream_t st) {
-    const int KP = p.maps * p.dp + 16 / (int)sizeof(T);
-    const size_t smem = (size_t)(QN * p.dp + QN * (kKeys + 4) + 4 * QN + kKeys) * 4 + (size_t)kKeys * (KP + p.vp) * sizeof(T);
-    const dim3 grid(p.splits, p.G * p.qgroups, p.M);
-    if (p.vdim <= kRowThreads) {
-        auto k = attention_rows_kernel<T, QN, 1>;
-        if (smem > 48 * 1024 && cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return check_launch();
-        launch_kernel(k, grid, dim3(kRowThreads), smem, st, p);
-    } else {
-        auto k = attention_rows_kernel<T, QN, 2>;
-        if (smem > 48 * 1024 && cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return check_launch();
-        launch_kernel(k, grid, dim3(kRowThreads), smem, st, p);
-    }
-    if (check_launch() != B200_OK) return B200_ECUDA;
-    launch_kernel(attention_merge_kernel<T>, dim3(p.H, p.M), dim3(kRowThreads), 0, st, p);
-    return check_launch();
+    return p.vdim <= kRowThreads ? launch_rows_c<T, QN, 1, false>(p, st) : launch_rows_c<T, QN, 2, false>(p, st);
+}
+template <typename T, int QN>
+int launch_rows_shared(AttnParams& p, cudaStream_t st) {
+    if (p.vdim <= 2 * kRowThreads) return launch_rows_c<T, QN, 2, true>(p, st);
+    if (p.vdim <= 4 * kRowThreads) return launch_rows_c<T, QN, 4, true>(p, st);
+    return B200_ELIMIT;
 }
 
 template <typename T>
@@ -512,9 +532,16 @@ int launch_rows_any(AttnParams& p, cudaStream_t st) {
     return launch_rows<T, 16>(p, st);
 }
 
-template <int VT, int MAPS>
+template <typename T>
+int launch_rows_latent(AttnParams& p, cudaStream_t st) {
+    if (p.hpg <= 4) return launch_rows_shared<T, 4>(p, st);
+    if (p.hpg <= 8) return launch_rows_shared<T, 8>(p, st);
+    return launch_rows_shared<T, 16>(p, st);
+}
+
+template <int VT, int MAPS, bool LATENT>
 int launch_prompt(const AttnParams& p, cudaStream_t st) {
-    auto k = attention_prompt_kernel<VT, MAPS>;
+    auto k = attention_prompt_kernel<VT, MAPS, LATENT>;
     const int KP = MAPS * p.dp + 8;
     const size_t smem = (size_t)(3 * kKeys * KP + 2 * kKeys * (VT * 16 + 8)) * 2;
     if (cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return check_launch();
@@ -522,12 +549,24 @@ int launch_prompt(const AttnParams& p, cudaStream_t st) {
     return check_launch();
 }
 
-template <int MAPS>
+template <int MAPS, bool LATENT>
 int launch_prompt_any(const AttnParams& p, cudaStream_t st) {
-    if (p.vp <= 32) return launch_prompt<2, MAPS>(p, st);
-    if (p.vp <= 64) return launch_prompt<4, MAPS>(p, st);
-    if (p.vp <= 96) return launch_prompt<6, MAPS>(p, st);
-    return launch_prompt<8, MAPS>(p, st);
+    if (p.vp <= 32) return launch_prompt<2, MAPS, LATENT>(p, st);
+    if (p.vp <= 64) return launch_prompt<4, MAPS, LATENT>(p, st);
+    if (p.vp <= 96) return launch_prompt<6, MAPS, LATENT>(p, st);
+    return launch_prompt<8, MAPS, LATENT>(p, st);
+}
+
+// Few-row passes of a latent layer: all heads read the same rows.  Heads of a CTA: what the shared memory holds.
+int launch_latent_rows(const b200_hybrid_model& m, const b200_hybrid_layer& l, AttnParams& p, int max_keys, cudaStream_t st) {
+    const int elem = act_bytes(m.act_type);
+    int most = 16;
+    while (most > 4 && rows_smem(p, most, elem, true) > kMaxSmem) most /= 2;
+    p.qgroups = (p.H + most - 1) / most;
+    p.hpg = (p.H + p.qgroups - 1) / p.qgroups;
+    p.splits = pick_splits(p.M, p.qgroups, (max_keys + p.tail + kKeys - 1) / kKeys);
+    if ((size_t)p.M * p.H * p.splits * (p.vp + 2) * 4 > m.attn_part_bytes) return B200_EWORKSPACE;
+    return m.act_type == B200_ACT_F32 ? launch_rows_latent<float>(p, st) : launch_rows_latent<bf16>(p, st);
 }
 
 }  // namespace
@@ -536,9 +575,9 @@ size_t attention_part_bytes(const b200_hybrid_model& m, int rows) {
     size_t most = 0;
     for (int i = 0; i < m.n_layers; i++) {
         const b200_hybrid_layer& l = m.layers[i];
-        if (l.mixer != B200_MIXER_ATTENTION) continue;
+        if (l.mixer != B200_MIXER_ATTENTION && l.mixer != B200_MIXER_LATENT) continue;
         const size_t r = rows > 592 ? rows : 592;        // rows * splits never exceeds it (pick_splits)
-        const size_t b = r * l.heads * l.maps * (round_up(l.vdim, 16) + 2) * 4;
+        const size_t b = r * l.heads * l.maps * (round_up(l.mixer == B200_MIXER_LATENT ? l.kv_rank : l.vdim, 16) + 2) * 4;
         most = b > most ? b : most;
     }
     return most;
@@ -548,14 +587,30 @@ int launch_attention(const b200_hybrid_model& m, const b200_hybrid_layer& l, con
                      cudaStream_t st) {
     AttnParams p{};
     char* cache = static_cast<char*>(ps.cache);
+    if (l.mixer == B200_MIXER_LATENT) {
+        const int cp = round_up(l.kv_rank, 16), rp = round_up(l.rot_dim, 16);
+        p.q = m.qb; p.part = m.attn_part; p.pos = ps.pos; p.tail_pos = ps.tail_pos; p.mask = ps.mask; p.prefix = ps.prefix;
+        p.M = ps.M; p.H = l.heads; p.maps = 1; p.window = l.window; p.keep = l.keep_first; p.tree = ps.tree;
+        p.tail = ps.tree ? ps.tail : 0; p.scale_log2 = l.scale * kLog2e; p.out_scale = 1.f; p.eps = m.eps;
+        if (latent_expands(m, l, ps)) {
+            p.G = l.heads; p.rp = rp; p.dim = l.dim; p.dp = round_up(l.dim, 16) + rp; p.vdim = l.vdim; p.vp = round_up(l.vdim, 16);
+            p.kc = m.kx; p.vc = m.vx; p.cap = m.x_rows; p.krot = cache + r.k_off + (size_t)cp * 2; p.krot_pitch = cp + rp;
+            p.q_pitch = l.heads * p.dp; p.out = m.ab; p.out_pitch = round_up(l.heads * l.vdim, 64); p.out_head = l.vdim;
+            return launch_prompt_any<1, true>(p, st);
+        }
+        p.G = 1; p.dim = p.dp = cp + rp; p.vdim = l.kv_rank; p.vp = cp; p.kc = cache + r.k_off; p.cap = ps.cache_rows;
+        p.q_pitch = l.heads * p.dp; p.out = m.ob; p.out_head = l.value.pitch; p.out_pitch = l.heads * l.value.pitch;
+        return launch_latent_rows(m, l, p, ps.max_keys, st);
+    }
     p.q = m.qb; p.kc = cache + r.k_off; p.vc = cache + r.v_off; p.gate = m.gb; p.out = m.ab; p.part = m.attn_part;
     p.pos = ps.pos; p.tail_pos = ps.tail_pos; p.mask = ps.mask; p.prefix = ps.prefix;
     p.M = ps.M; p.H = l.heads; p.G = l.kv_heads; p.maps = l.maps; p.dim = l.dim; p.dp = round_up(l.dim, 16); p.vdim = l.vdim;
     p.vp = round_up(l.vdim, 16); p.cap = ps.cache_rows; p.window = l.window; p.keep = l.keep_first; p.tree = ps.tree;
     p.tail = ps.tree ? ps.tail : 0; p.q_pitch = l.heads * l.maps * p.dp; p.out_pitch = round_up(l.heads * l.vdim, 64);
+    p.out_head = l.vdim;
     p.scale_log2 = l.scale * kLog2e; p.lambda = l.lambda; p.out_scale = l.out_scale; p.eps = m.eps;
     if (m.act_type == B200_ACT_BF16 && !ps.tree && ps.M > 16 && p.dp <= 128 && p.vp <= 128)
-        return l.maps == 2 ? launch_prompt_any<2>(p, st) : launch_prompt_any<1>(p, st);
+        return l.maps == 2 ? launch_prompt_any<2, false>(p, st) : launch_prompt_any<1, false>(p, st);
     pick_groups(p.H / p.G, p.maps, &p.hpg, &p.qgroups);
     long long keys = (long long)l.window + l.keep_first;
     if (keys > ps.max_keys) keys = ps.max_keys;

@@ -1,0 +1,424 @@
+// Gated delta rule of the hybrid decoders, one decay per head and key channel:
+//     S <- g * S (rows);   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q,
+// q and k unit vectors; q, k, v come out of short causal convolutions with silu.  Everything that enters the recurrence is
+// fp32, the state [heads][vdim][dim] is carried in the request's cache, as are the convolutions' last inputs.
+//
+//   conv_kernel    convolution, silu and unit norm: a warp per head of q, k or v and block of rows.
+//   scan_kernel    CTA = (head, 32 state columns); 8 lanes share a column and hold its rows in registers (packed pairs), so the
+//                  read-out of k before the write takes three shuffles; tokens come in blocks through shared memory and the
+//                  lanes' parts of the outputs are added for 8 tokens at once.  Three forms:
+//                    chain   the pass's rows in order; the new state and convolution inputs are written back;
+//                    tree    a CTA per row replays the row's path from the state, nothing is written back;
+//                    commit  pending rows are replayed and written back, no output.
+#include "scan.cuh"
+
+namespace b200 {
+namespace hybrid {
+namespace {
+
+constexpr int kThreads = 256;
+constexpr int kConvRows = 8;             // chain rows of a warp
+constexpr int kLanes = 8;                // lanes of a state column
+constexpr int kMaxDim = 256;
+enum : int { kChain = 0, kTree = 1, kCommit = 2 };
+
+struct ConvParams {
+    const void* in;          // chain: [M][pitch]; tree: pending rows [64][pitch]
+    const void* state;       // [taps - 1][pitch] committed inputs, oldest first
+    const float* w;          // [taps][channels]
+    const unsigned long long* mask;
+    float* q;                // [M][G * d]
+    float* k;                // [M][G * d], tree: pending rows from write_off on
+    void* v;                 // [M][H * dv], likewise
+    int M, G, H, d, dv, taps, pitch, channels, write_off;
+};
+
+// A lane holds NI vectors of V neighbouring channels.
+template <typename T, int V> __device__ __forceinline__ void ld_vec(float (&r)[V], const T* p) {
+    if constexpr (V == 4 && sizeof(T) == 2) {
+        const uint2 u = *reinterpret_cast<const uint2*>(p);
+        r[0] = __uint_as_float(u.x << 16);
+        r[1] = __uint_as_float(u.x & 0xffff0000u);
+        r[2] = __uint_as_float(u.y << 16);
+        r[3] = __uint_as_float(u.y & 0xffff0000u);
+    } else {
+#pragma unroll
+        for (int e = 0; e < V; e++) r[e] = to_f32<T>(p[e]);
+    }
+}
+
+template <typename T, int V, int NI, bool TREE>
+__global__ void __launch_bounds__(kThreads) conv_kernel(const ConvParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    constexpr int R = TREE ? 1 : kConvRows;
+    __shared__ const T* s_src[B200_HYBRID_MAX_TAPS];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = blockIdx.y * R, rows = min(R, p.M - r0);
+    const T* in = static_cast<const T*>(p.in);
+    const T* state = static_cast<const T*>(p.state);
+    if (TREE) {                              // the row's inputs along its path: ancestors (set bits of its mask), then committed ones
+        if (threadIdx.x == 0) {
+            const int self = p.write_off + r0;
+            unsigned long long anc = p.mask[r0] & ((1ull << self) - 1ull);
+            int have = 0;
+            s_src[p.taps - 1] = in + (size_t)self * p.pitch;
+            for (int j = p.taps - 2; j >= 0; j--) {
+                if (anc != 0ull) {
+                    const int a = 63 - __clzll((long long)anc);
+                    anc &= ~(1ull << a);
+                    have++;
+                    s_src[j] = in + (size_t)a * p.pitch;
+                } else {
+                    s_src[j] = state + (size_t)(j + have) * p.pitch;
+                }
+            }
+        }
+        __syncthreads();
+    }
+    const int unit = blockIdx.x * (kThreads / 32) + warp;
+    if (unit >= 2 * p.G + p.H) return;
+    const bool value = unit >= 2 * p.G;
+    const int n = value ? p.dv : p.d, c0 = value ? 2 * p.G * p.d + (unit - 2 * p.G) * p.dv : unit * p.d;
+    float acc[R][NI][V];
+#pragma unroll
+    for (int r = 0; r < R; r++)
+#pragma unroll
+        for (int i = 0; i < NI; i++)
+#pragma unroll
+            for (int e = 0; e < V; e++) acc[r][i][e] = 0.f;
+    for (int j = 0; j < p.taps; j++) {
+#pragma unroll
+        for (int i = 0; i < NI; i++) {
+            const int c = (lane + 32 * i) * V;
+            if (c >= n) continue;
+            float w[V];
+#pragma unroll
+            for (int e = 0; e < V; e++) w[e] = p.w[(size_t)j * p.channels + c0 + c + e];
+#pragma unroll
+            for (int r = 0; r < R; r++) {
+                if (r >= rows) continue;
+                const int row = r0 + r - (p.taps - 1) + j;
+                const T* src = TREE ? s_src[j] : (row >= 0 ? in + (size_t)row * p.pitch : state + (size_t)(row + p.taps - 1) * p.pitch);
+                float x[V];
+                ld_vec<T, V>(x, src + c0 + c);
+#pragma unroll
+                for (int e = 0; e < V; e++) acc[r][i][e] = fmaf(w[e], x[e], acc[r][i][e]);
+            }
+        }
+    }
+    const float scale = unit < p.G ? rsqrtf((float)p.d) : 1.f;
+#pragma unroll
+    for (int r = 0; r < R; r++) {
+        if (r >= rows) continue;
+        const int m = r0 + r;
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; i++)
+#pragma unroll
+            for (int e = 0; e < V; e++) {
+                const float z = acc[r][i][e];        // (channels past the head are zero)
+                acc[r][i][e] = z * sigmoid_f(z);
+                ss = fmaf(acc[r][i][e], acc[r][i][e], ss);
+            }
+        float f = 1.f;
+        if (!value) f = rsqrtf(warp_sum(ss) + 1e-6f) * scale;
+#pragma unroll
+        for (int i = 0; i < NI; i++) {
+            const int c = (lane + 32 * i) * V;
+            if (c >= n) continue;
+            if (value) {
+                T* dst = static_cast<T*>(p.v) + ((size_t)m * p.H + unit - 2 * p.G) * p.dv + c;
+#pragma unroll
+                for (int e = 0; e < V; e++) dst[e] = from_f32<T>(acc[r][i][e]);
+            } else {
+                float* dst = (unit < p.G ? p.q : p.k) + ((size_t)m * p.G + (unit < p.G ? unit : unit - p.G)) * p.d + c;
+                if constexpr (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(acc[r][i][0] * f, acc[r][i][1] * f, acc[r][i][2] * f, acc[r][i][3] * f);
+                else dst[0] = acc[r][i][0] * f;
+            }
+        }
+    }
+}
+
+struct ScanParams {
+    const float* q;          // [M][G * d]
+    const float* k;          // chain: [M][G * d]; tree, commit: pending rows
+    const float* g;          // [..][H * d]
+    const float* beta;       // [..][H]
+    const void* v;           // [..][H * dv]
+    float* state;            // [H][dv][d]
+    float* o;                // [M][H * dv]
+    const void* in;          // convolution inputs [..][pitch]
+    void* conv_state;        // [taps - 1][pitch]
+    const unsigned long long* mask;
+    const int* count;        // commit: as b200_hybrid_commit
+    const int* rows;
+    int M, H, G, d, dv, taps, pitch, channels, tree_rows;
+};
+
+__device__ __forceinline__ void cp_async4(uint32_t dst, const void* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(dst), "l"(src) : "memory");
+}
+
+// Sum of v[i] over groups of 8 neighbouring lanes, for 8 values at once: lane i of a group gets the total of v[i].
+__device__ __forceinline__ float transpose_sum8(float (&v)[8], int lane) {
+#pragma unroll
+    for (int s = 4; s > 0; s >>= 1)
+#pragma unroll
+        for (int i = 0; i < s; i++) {
+            const bool up = (lane & s) != 0;
+            const float keep = up ? v[i + s] : v[i], send = up ? v[i] : v[i + s];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, send, s);
+        }
+    return v[0];
+}
+
+template <int RPL> __host__ __device__ constexpr int scan_block() { return RPL == 32 ? 8 : 16; }      // tokens of a shared-memory block
+
+template <typename T, int RPL, int MODE>         // state rows of a lane
+__global__ void __launch_bounds__(kThreads) scan_kernel(const ScanParams p) {
+    pdl_launch_dependents();
+    constexpr int D = kLanes * RPL, TB = scan_block<RPL>(), STAGES = 2;
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    float* sg = reinterpret_cast<float*>(smem_raw);      // [STAGES][TB][D]
+    float* sk = sg + STAGES * TB * D;
+    float* sq = sk + STAGES * TB * D;
+    float* sb = sq + STAGES * TB * D;                    // [STAGES][TB]
+    T* sv = reinterpret_cast<T*>(sb + STAGES * TB);      // [STAGES][TB][32]
+    __shared__ int s_row[B200_HYBRID_PENDING];
+    const int h = blockIdx.y, c0 = blockIdx.x * 32, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int kh = h / (p.H / p.G), d = p.d, dv = p.dv, m = blockIdx.z;
+    const int ncol = min(32, dv - c0), col = c0 + warp * 4 + (lane >> 3), j = lane & 7;
+    const bool wide = d % 4 == 0, wide_v = dv * (int)sizeof(T) % 16 == 0;
+    // what the copies never write stays zero: rows past the head's width, columns past its values, queries that are not asked for
+    for (int i = tid; i < STAGES * TB * D; i += kThreads) { sg[i] = 0.f; sk[i] = 0.f; sq[i] = 0.f; }
+    for (int i = tid; i < STAGES * TB * 32; i += kThreads) sv[i] = from_f32<T>(0.f);
+    pdl_wait();
+    int n = p.M;
+    if (MODE == kTree) {
+        const unsigned long long path = p.mask[m];
+        n = __popcll(path);
+        if (tid < B200_HYBRID_PENDING && ((path >> tid) & 1ull)) s_row[__popcll(path & ((1ull << tid) - 1ull))] = tid;
+    } else if (MODE == kCommit) {
+        n = min(max(p.count[0] + 1, 0), B200_HYBRID_PENDING);
+        for (int i = tid; i < n; i += kThreads) {
+            int s = i == 0 || p.rows == nullptr ? i : p.rows[i];
+            if (s < 0) s += p.tree_rows;
+            s_row[i] = min(max(s, 0), B200_HYBRID_PENDING - 1);
+        }
+    }
+    __syncthreads();
+    auto row_of = [&](int t) { return MODE == kChain ? t : s_row[t]; };
+    auto fetch = [&](int b) {
+        const int st = (b & 1) * TB, t0 = b * TB;
+        for (int t = warp; t < TB && t0 + t < n; t += kThreads / 32) {
+            const int row = row_of(t0 + t);
+            fetch_row(sg + (st + t) * D, p.g + ((size_t)row * p.H + h) * d, d, wide, lane);
+            fetch_row(sk + (st + t) * D, p.k + ((size_t)row * p.G + kh) * d, d, wide, lane);
+            if (MODE == kChain) fetch_row(sq + (st + t) * D, p.q + ((size_t)row * p.G + kh) * d, d, wide, lane);
+            if (MODE == kTree && t0 + t == n - 1) fetch_row(sq + (st + t) * D, p.q + ((size_t)m * p.G + kh) * d, d, wide, lane);
+            fetch_row(sv + (st + t) * 32, static_cast<const T*>(p.v) + ((size_t)row * p.H + h) * dv + c0, ncol, wide_v, lane);
+            if (lane == 0) cp_async4(smem_u32(sb + st + t), p.beta + (size_t)row * p.H + h);
+        }
+        asm volatile("cp.async.commit_group;\n" ::: "memory");
+    };
+    fetch(0);
+    unsigned long long S[RPL / 2];                       // state rows 32 i + 4 j + (0 .. 3) of the column, in pairs
+    float* sbase = p.state + ((size_t)h * dv + min(col, dv - 1)) * d;
+#pragma unroll
+    for (int i = 0; i < RPL / 4; i++) {
+        const int r = 32 * i + 4 * j;
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (wide) {
+            if (r < d) x = *reinterpret_cast<const float4*>(sbase + r);
+        } else {
+            if (r < d) x.x = sbase[r];
+            if (r + 1 < d) x.y = sbase[r + 1];
+            if (r + 2 < d) x.z = sbase[r + 2];
+            if (r + 3 < d) x.w = sbase[r + 3];
+        }
+        S[2 * i] = pack2(x.x, x.y);
+        S[2 * i + 1] = pack2(x.z, x.w);
+    }
+    const int nb = (n + TB - 1) / TB;
+    for (int b = 0; b < nb; b++) {
+        const int st = (b & 1) * TB, t0 = b * TB;
+        asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+        __syncthreads();                                 // this block is here, the one before has been read
+        if (b + 1 < nb) fetch(b + 1);
+#pragma unroll 1
+        for (int tg = 0; tg < TB && t0 + tg < n; tg += 8) {
+            const int nt = min(8, n - t0 - tg);
+            float y[8];                                  // this lane's rows
+#pragma unroll
+            for (int t = 0; t < 8; t++) {
+                y[t] = 0.f;
+                if (t >= nt) continue;
+                const int at = st + tg + t;
+                const ulonglong2* g4 = reinterpret_cast<const ulonglong2*>(sg + at * D + 4 * j);
+                const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(sk + at * D + 4 * j);
+                const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(sq + at * D + 4 * j);
+                const float v = to_f32<T>(sv[at * 32 + warp * 4 + (lane >> 3)]), beta = sb[at];
+                unsigned long long k2[RPL / 2], a0 = 0ull, a1 = 0ull;
+#pragma unroll
+                for (int i = 0; i < RPL / 4; i++) {
+                    const ulonglong2 g = g4[8 * i], k = k4[8 * i];
+                    k2[2 * i] = k.x;
+                    k2[2 * i + 1] = k.y;
+                    S[2 * i] = mul2(S[2 * i], g.x);
+                    S[2 * i + 1] = mul2(S[2 * i + 1], g.y);
+                    a0 = fma2(k.x, S[2 * i], a0);
+                    a1 = fma2(k.y, S[2 * i + 1], a1);
+                }
+                const float2 x0 = unpack2(a0), x1 = unpack2(a1);
+                float r = (x0.x + x0.y) + (x1.x + x1.y);
+#pragma unroll
+                for (int o = 1; o < kLanes; o <<= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
+                const float u = beta * (v - r);
+                const unsigned long long u2 = pack2(u, u);
+                a0 = 0ull;
+                a1 = 0ull;
+#pragma unroll
+                for (int i = 0; i < RPL / 4; i++) {
+                    S[2 * i] = fma2(k2[2 * i], u2, S[2 * i]);
+                    S[2 * i + 1] = fma2(k2[2 * i + 1], u2, S[2 * i + 1]);
+                    if (MODE != kCommit) {
+                        const ulonglong2 q = q4[8 * i];
+                        a0 = fma2(q.x, S[2 * i], a0);
+                        a1 = fma2(q.y, S[2 * i + 1], a1);
+                    }
+                }
+                if (MODE != kCommit) {
+                    const float2 z0 = unpack2(a0), z1 = unpack2(a1);
+                    y[t] = (z0.x + z0.y) + (z1.x + z1.y);
+                }
+            }
+            if (MODE == kCommit) continue;
+            const float out = transpose_sum8(y, lane);
+            const int t = t0 + tg + j;
+            if (MODE == kChain) {
+                if (j < nt && col < dv) p.o[((size_t)t * p.H + h) * dv + col] = out;
+            } else if (t == n - 1 && col < dv) {
+                p.o[((size_t)m * p.H + h) * dv + col] = out;
+            }
+        }
+    }
+    if (MODE == kTree) return;
+    if (col < dv) {
+#pragma unroll
+        for (int i = 0; i < RPL / 4; i++) {
+            const int r = 32 * i + 4 * j;
+            const float2 x = unpack2(S[2 * i]), y = unpack2(S[2 * i + 1]);
+            if (wide) {
+                if (r < d) *reinterpret_cast<float4*>(sbase + r) = make_float4(x.x, x.y, y.x, y.y);
+            } else {
+                if (r < d) sbase[r] = x.x;
+                if (r + 1 < d) sbase[r + 1] = x.y;
+                if (r + 2 < d) sbase[r + 2] = y.x;
+                if (r + 3 < d) sbase[r + 3] = y.y;
+            }
+        }
+    }
+    // the convolutions' last inputs, channels over all CTAs
+    const int prev = p.taps - 1;
+    const T* in = static_cast<const T*>(p.in);
+    T* cs = static_cast<T*>(p.conv_state);
+    if (prev > 0) {
+        for (int c = (blockIdx.y * gridDim.x + blockIdx.x) * kThreads + tid; c < p.channels; c += gridDim.x * gridDim.y * kThreads) {
+            T nv[B200_HYBRID_MAX_TAPS];
+#pragma unroll
+            for (int e = 0; e < B200_HYBRID_MAX_TAPS; e++)
+                if (e < prev) {
+                    const int i = n - prev + e;
+                    nv[e] = i >= 0 ? in[(size_t)row_of(i) * p.pitch + c] : cs[(size_t)(i + prev) * p.pitch + c];
+                }
+#pragma unroll
+            for (int e = 0; e < B200_HYBRID_MAX_TAPS; e++)
+                if (e < prev) cs[(size_t)e * p.pitch + c] = nv[e];
+        }
+    }
+}
+
+template <typename T, int RPL, int MODE>
+int launch_scan_r(const ScanParams& p, int rows, cudaStream_t st) {
+    constexpr int TB = scan_block<RPL>(), D = kLanes * RPL;
+    const size_t smem = 2 * TB * ((size_t)3 * D * 4 + 4 + 32 * sizeof(T));
+    auto k = scan_kernel<T, RPL, MODE>;
+    if (smem > 40 * 1024 && cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return check_launch();
+    launch_kernel(k, dim3((p.dv + 31) / 32, p.H, rows), dim3(kThreads), smem, st, p);
+    return check_launch();
+}
+template <typename T, int MODE>
+int launch_scan(const ScanParams& p, int rows, cudaStream_t st) {
+    if (p.d <= 64) return launch_scan_r<T, 8, MODE>(p, rows, st);
+    if (p.d <= 128) return launch_scan_r<T, 16, MODE>(p, rows, st);
+    return launch_scan_r<T, 32, MODE>(p, rows, st);
+}
+
+template <typename T, int V, int NI>
+void launch_conv_v(const ConvParams& p, bool tree, cudaStream_t st) {
+    const int units = (2 * p.G + p.H + kThreads / 32 - 1) / (kThreads / 32);
+    if (tree) launch_kernel(conv_kernel<T, V, NI, true>, dim3(units, p.M), dim3(kThreads), 0, st, p);
+    else launch_kernel(conv_kernel<T, V, NI, false>, dim3(units, (p.M + kConvRows - 1) / kConvRows), dim3(kThreads), 0, st, p);
+}
+
+template <typename T>
+int delta(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_run& r, const b200_hybrid_pass& ps, cudaStream_t st) {
+    char* pend = static_cast<char*>(m.pending);
+    char* cache = static_cast<char*>(ps.cache);
+    const size_t off = ps.write_off;
+    const int nk = l.kv_heads * l.dim, nv = l.heads * l.vdim;
+    ConvParams c{};
+    c.in = ps.tree ? pend + r.pend_c : static_cast<char*>(m.cb);
+    c.state = cache + r.mix_off; c.w = l.mix_conv; c.mask = ps.mask; c.q = m.q32;
+    c.k = ps.tree ? reinterpret_cast<float*>(pend + r.pend_k) + off * nk : m.k32;
+    c.v = ps.tree ? static_cast<void*>(reinterpret_cast<T*>(pend + r.pend_v) + off * nv) : m.vb;
+    c.M = ps.M; c.G = l.kv_heads; c.H = l.heads; c.d = l.dim; c.dv = l.vdim; c.taps = l.conv_taps; c.pitch = delta_pitch(l);
+    c.channels = delta_channels(l); c.write_off = ps.write_off;
+    const int most = l.dim > l.vdim ? l.dim : l.vdim;
+    if (l.dim % 4 || l.vdim % 4) launch_conv_v<T, 1, 8>(c, ps.tree, st);
+    else if (most <= 128) launch_conv_v<T, 4, 1>(c, ps.tree, st);
+    else launch_conv_v<T, 4, 2>(c, ps.tree, st);
+    if (check_launch() != B200_OK) return B200_ECUDA;
+    ScanParams s{};
+    s.q = m.q32; s.state = reinterpret_cast<float*>(cache + r.state_off); s.o = m.o32; s.in = c.in; s.conv_state = cache + r.mix_off;
+    s.k = ps.tree ? reinterpret_cast<const float*>(pend + r.pend_k) : m.k32;
+    s.g = ps.tree ? reinterpret_cast<const float*>(pend + r.pend_g) : m.gf;
+    s.beta = ps.tree ? reinterpret_cast<const float*>(pend + r.pend_b) : m.beta;
+    s.v = ps.tree ? static_cast<const void*>(pend + r.pend_v) : m.vb;
+    s.mask = ps.mask; s.M = ps.M; s.H = l.heads; s.G = l.kv_heads; s.d = l.dim; s.dv = l.vdim; s.taps = l.conv_taps; s.pitch = c.pitch;
+    s.channels = c.channels;
+    const int rc = ps.tree ? launch_scan<T, kTree>(s, ps.M, st) : launch_scan<T, kChain>(s, 1, st);
+    return rc != B200_OK ? rc : launch_head_norm(m, l, ps.M, m.gb, st);
+}
+
+template <typename T>
+int delta_commit(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_run& r, char* cache, const int* count, const int* rows,
+                 int tree_rows, cudaStream_t st) {
+    char* pend = static_cast<char*>(m.pending);
+    ScanParams s{};
+    s.state = reinterpret_cast<float*>(cache + r.state_off); s.in = pend + r.pend_c; s.conv_state = cache + r.mix_off;
+    s.k = reinterpret_cast<const float*>(pend + r.pend_k);
+    s.g = reinterpret_cast<const float*>(pend + r.pend_g);
+    s.beta = reinterpret_cast<const float*>(pend + r.pend_b);
+    s.v = pend + r.pend_v;
+    s.count = count; s.rows = rows; s.tree_rows = tree_rows;
+    s.H = l.heads; s.G = l.kv_heads; s.d = l.dim; s.dv = l.vdim; s.taps = l.conv_taps; s.pitch = delta_pitch(l); s.channels = delta_channels(l);
+    return launch_scan<T, kCommit>(s, 1, st);
+}
+
+}  // namespace
+
+int launch_delta(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_run& r, const b200_hybrid_pass& p, cudaStream_t st) {
+    if (l.dim > kMaxDim || l.vdim > kMaxDim) return B200_ELIMIT;
+    return m.act_type == B200_ACT_F32 ? delta<float>(m, l, r, p, st) : delta<bf16>(m, l, r, p, st);
+}
+
+int launch_delta_commit(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_run& r, void* cache, const int* count,
+                        const int* rows, int tree_rows, cudaStream_t st) {
+    if (l.dim > kMaxDim || l.vdim > kMaxDim) return B200_ELIMIT;
+    char* c = static_cast<char*>(cache);
+    return m.act_type == B200_ACT_F32 ? delta_commit<float>(m, l, r, c, count, rows, tree_rows, st) : delta_commit<bf16>(m, l, r, c, count, rows, tree_rows, st);
+}
+
+}  // namespace hybrid
+}  // namespace b200

@@ -47,10 +47,47 @@ struct Geo {
 struct GemmParams {
     CUtensorMap wmap, xmap;
     Epi epi;
-    int N, kblocks, ntiles, ttiles;   // 128-row tiles, token tiles
+    int kblocks, ntiles, ttiles;      // 128-row tiles of all groups, token tiles
+    int gtiles, gn, xg;               // tiles, rows and x columns of a group
     int ksplit;                       // CTAs of a cluster that share a tile's K range (1: none)
+    int groups;
+    const int* offsets;               // expert stacks: first token row of every group
     int* error;
 };
+
+// What a tile multiplies: weight row, x column and token row of its corner, output column of its first row.
+struct Tile {
+    int wrow, xcol, tok0, tokend, col0, rows;
+};
+__device__ __forceinline__ Tile tile_at(const GemmParams& p, int t, int nt) {
+    Tile r;
+    const int w = t / p.ttiles, g = w / p.gtiles, lt = w - g * p.gtiles;
+    r.wrow = w * kTileRows;
+    r.xcol = g * p.xg;
+    r.tok0 = (t - w * p.ttiles) * nt;
+    r.tokend = p.epi.M;
+    r.col0 = g * p.gn + lt * kTileRows;
+    r.rows = p.gn - lt * kTileRows;
+    return r;
+}
+// Expert stacks: tile0[g] token tiles before group g; a group's tiles are ordered token tile fastest.
+__device__ __forceinline__ Tile expert_tile_at(const GemmParams& p, const int* off, const int* tile0, int t, int nt) {
+    Tile r;
+    int lo = 0, hi = p.groups - 1;
+    while (lo < hi) {
+        const int mid = (lo + hi + 1) >> 1;
+        if (tile0[mid] * p.gtiles <= t) lo = mid;
+        else hi = mid - 1;
+    }
+    const int rem = t - tile0[lo] * p.gtiles, tt = tile0[lo + 1] - tile0[lo], lt = rem / tt;
+    r.wrow = (lo * p.gtiles + lt) * kTileRows;
+    r.xcol = 0;
+    r.tok0 = off[lo] + (rem - lt * tt) * nt;
+    r.tokend = off[lo + 1];
+    r.col0 = lt * kTileRows;
+    r.rows = p.gn - lt * kTileRows;
+    return r;
+}
 
 __device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
     asm volatile(
@@ -81,7 +118,7 @@ __device__ __forceinline__ float ld_cluster_f32(uint32_t saddr, uint32_t rank) {
     return v;
 }
 
-template <int NT>
+template <int NT, bool EXPERTS>
 __global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const __grid_constant__ GemmParams p) {
     using G = Geo<NT>;
     extern __shared__ unsigned char smem_raw[];
@@ -93,14 +130,16 @@ __global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const _
     uint64_t* accempty = accfull + G::NACC;
     __shared__ uint32_t s_tmem;
     __shared__ int s_abort;
+    __shared__ int s_off[EXPERTS ? B200_HYBRID_MAX_EXPERTS + 1 : 1], s_tile0[EXPERTS ? B200_HYBRID_MAX_EXPERTS + 1 : 1];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int ks = p.ksplit;
     const uint32_t rank = ks > 1 ? cluster_rank() : 0u;
     // K blocks of this CTA, output tiles of this CTA
     const int kb0 = (int)((long long)p.kblocks * rank / ks), kb1 = (int)((long long)p.kblocks * (rank + 1) / ks);
     const int nk = kb1 - kb0;
-    const int tiles = p.ntiles * p.ttiles;
+    int tiles = EXPERTS ? 0 : p.ntiles * p.ttiles;
     const int tile0 = blockIdx.x / ks, tile_step = gridDim.x / ks;
+    auto tile_of = [&](int t) { return EXPERTS ? expert_tile_at(p, s_off, s_tile0, t, NT) : tile_at(p, t, NT); };
 
     if (threadIdx.x == 0) {
         s_abort = 0;
@@ -118,9 +157,30 @@ __global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const _
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(smem_u32(&s_tmem)), "n"(G::TMEM_COLS) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
     }
+    if (EXPERTS) {
+        pdl_wait();
+        for (int e = threadIdx.x; e <= p.groups; e += kThreads) s_off[e] = p.offsets[e];
+        __syncthreads();
+        if (warp == 0) {                                    // token tiles before each group
+            int before = 0;
+            for (int e0 = 0; e0 < p.groups; e0 += 32) {
+                const int e = e0 + lane;
+                int n = e < p.groups ? (s_off[e + 1] - s_off[e] + NT - 1) / NT : 0;
+#pragma unroll
+                for (int o = 1; o < 32; o <<= 1) {
+                    const int u = __shfl_up_sync(0xffffffffu, n, o);
+                    if (lane >= o) n += u;
+                }
+                if (e < p.groups) s_tile0[e + 1] = before + n;
+                before += __shfl_sync(0xffffffffu, n, 31);
+            }
+            if (lane == 0) s_tile0[0] = 0;
+        }
+    }
     asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+    if (EXPERTS) tiles = s_tile0[p.groups] * p.gtiles;
     const uint32_t tmem = s_tmem;
     volatile int* abort_flag = &s_abort;
     uint32_t issued = 0;                                    // producer: stages whose copies were issued
@@ -132,7 +192,7 @@ __global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const _
             // weights of the first stages, before anything of an earlier kernel is read
             uint32_t pre = 0;
             if (tile0 < tiles) {
-                const int row = (tile0 / p.ttiles) * kTileRows;
+                const int row = tile_of(tile0).wrow;
                 pre = nk < G::STAGES ? nk : G::STAGES;
                 for (uint32_t s = 0; s < pre; s++) {
                     mbar_expect_tx(smem_u32(full + s), G::STAGE);
@@ -143,7 +203,7 @@ __global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const _
             pdl_launch_dependents();
             bool ok = true;
             for (int t = tile0; t < tiles && ok; t += tile_step) {
-                const int row = (t / p.ttiles) * kTileRows, tok = (t % p.ttiles) * NT;
+                const Tile at = tile_of(t);
                 for (int kb = kb0; kb < kb1; kb++, n++) {
                     const uint32_t s = n % G::STAGES, use = n / G::STAGES;
                     if (use > 0) {
@@ -153,9 +213,9 @@ __global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const _
                     const uint32_t bar = smem_u32(full + s), dst = smem_u32(smem + s * G::STAGE);
                     if (n >= pre) {
                         mbar_expect_tx(bar, G::STAGE);
-                        tma_load_2d(dst, &p.wmap, kb * kTileK, row, bar);
+                        tma_load_2d(dst, &p.wmap, kb * kTileK, at.wrow, bar);
                     }
-                    tma_load_2d(dst + kWBytes, &p.xmap, kb * kTileK, tok, bar);
+                    tma_load_2d(dst + kWBytes, &p.xmap, at.xcol + kb * kTileK, at.tok0, bar);
                     issued = n + 1;
                 }
             }
@@ -215,15 +275,17 @@ __global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const _
             ok = __all_sync(0xffffffffu, !*abort_flag && gwait(smem_u32(accfull + ab), ause & 1u));
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-            const int tok0 = (t % p.ttiles) * NT;
+            const Tile at = tile_of(t);
+            const int tok0 = at.tok0;
             const uint32_t taddr = tmem + ab * G::ACC_COLS + ((uint32_t)(warp * 32) << 16);
             const int r = warp * 32 + lane;
             ColumnOut<bf16> out;
-            if (ks == 1) out.init(p.epi, (t / p.ttiles) * kTileRows + r);
+            const bool gated = p.epi.gate.kind != 0;
+            if (ks == 1 && !gated) out.init(p.epi, r < at.rows ? at.col0 + r : -1);
             float* part = reinterpret_cast<float*>(smem);          // split: [token][128], over the drained ring
 #pragma unroll 1
             for (int c = 0; c < NT; c += 16) {
-                if (tok0 + c >= p.epi.M) break;
+                if (tok0 + c >= at.tokend) break;
                 uint32_t v[16];
                 asm volatile(
                     "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];\n"
@@ -235,8 +297,10 @@ __global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const _
                 if (ks > 1) {
 #pragma unroll
                     for (int i = 0; i < 16; i++) part[(c + i) * kTileRows + r] = __uint_as_float(v[i]);
+                } else if (gated) {
+                    store_gated_rows<bf16, 16>(p.epi, at.col0 + r, r < at.rows, tok0 + c, at.tokend - tok0 - c, v);
                 } else {
-                    out.store_rows<16>(tok0 + c, p.epi.M - tok0 - c, v);
+                    out.store_rows<16>(tok0 + c, at.tokend - tok0 - c, v);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
@@ -252,13 +316,11 @@ __global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const _
         __syncthreads();
         cluster_sync_all();
         if (tile0 < tiles && !*abort_flag) {
+            const Tile at = tile_of(tile0);
             const int r0 = kTileRows * (int)rank / ks, share = kTileRows * ((int)rank + 1) / ks - r0;
-            const int tok0 = (tile0 % p.ttiles) * NT, ntok = min(NT, p.epi.M - tok0);
+            const int tok0 = at.tok0, ntok = min(NT, at.tokend - tok0);
             const uint32_t part = smem_u32(smem);
-            for (int i = threadIdx.x; i < share * ntok; i += kThreads) {
-                const int c = i / share, r = r0 + i - c * share;
-                ColumnOut<bf16> out;
-                out.init(p.epi, (tile0 / p.ttiles) * kTileRows + r);
+            auto total = [&](int c, int r) {
                 float v[kMaxSplit];
 #pragma unroll
                 for (int q = 0; q < kMaxSplit; q++)
@@ -266,7 +328,24 @@ __global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const _
                 float a = 0.f;
 #pragma unroll
                 for (int q = 0; q < kMaxSplit; q++) a += v[q];
-                out.store(tok0 + c, a);
+                return a;
+            };
+            if (p.epi.gate.kind != 0) {
+                for (int i = threadIdx.x; i < share / 2 * ntok; i += kThreads) {
+                    const int c = i / (share / 2), r = r0 + 2 * (i - c * (share / 2)), n = at.col0 + r, m = tok0 + c;
+                    if (r >= at.rows) continue;
+                    const float sc = p.epi.row_scale != nullptr ? p.epi.row_scale[m] : 1.f;
+                    float g = total(c, r) * sc, u = total(c, r + 1) * sc;
+                    if (p.epi.gate_bias != nullptr) { g += p.epi.gate_bias[n]; u += p.epi.gate_bias[n + 1]; }
+                    static_cast<bf16*>(p.epi.seg[0].dst)[(long long)m * p.epi.seg[0].row_stride + (n >> 1)] = __float2bfloat16_rn(gated_f(p.epi.gate, g, u));
+                }
+            } else {
+                for (int i = threadIdx.x; i < share * ntok; i += kThreads) {
+                    const int c = i / share, r = r0 + i - c * share;
+                    ColumnOut<bf16> out;
+                    out.init(p.epi, r < at.rows ? at.col0 + r : -1);
+                    out.store(tok0 + c, total(c, r));
+                }
             }
         }
         cluster_sync_all();                                        // no CTA leaves while its shared memory is read
@@ -316,34 +395,45 @@ int sm_count() {
     return sms;
 }
 
-template <int NT>
-int launch_gemm(const b200_linear& lin, const void* x, int x_rows, const Epi& epi, int* error, cudaStream_t st) {
+template <int NT, bool EXPERTS>
+int launch_gemm(const b200_linear& lin, const void* x, int x_pitch, int x_rows, const Epi& epi, int rows, const int* offsets, int* error, cudaStream_t st) {
     using G = Geo<NT>;
-    auto kern = gemm_kernel<NT>;
+    auto kern = gemm_kernel<NT, EXPERTS>;
     static bool attr = false;
     if (!attr) {
         if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, G::SMEM) != cudaSuccess) return check_launch();
         attr = true;
     }
     GemmParams p;
-    int rc = make_map(&p.wmap, lin.w, lin.pitch, round_up(lin.n, kTileRows), kTileRows);
-    if (rc == B200_OK) rc = make_map(&p.xmap, x, lin.pitch, x_rows, NT);
+    const int groups = lin.groups > 1 ? lin.groups : 1;
+    int rc = make_map(&p.wmap, lin.w, lin.pitch, groups * round_up(lin.n, kTileRows), kTileRows);
+    if (rc == B200_OK) rc = make_map(&p.xmap, x, x_pitch, x_rows, NT);
     if (rc != B200_OK) return rc;
     p.epi = epi;
-    p.N = lin.n;
     p.kblocks = lin.pitch / kTileK;
-    p.ntiles = (lin.n + kTileRows - 1) / kTileRows;
-    p.ttiles = (epi.M + NT - 1) / NT;
+    p.gtiles = (lin.n + kTileRows - 1) / kTileRows;
+    p.gn = lin.n;
+    p.xg = lin.pitch;
+    p.groups = groups;
+    p.offsets = offsets;
+    p.ntiles = groups * p.gtiles;
+    p.ttiles = (rows + NT - 1) / NT;
     p.error = error;
     p.ksplit = 1;
     const int sms = sm_count(), tiles = p.ntiles * p.ttiles;
-    if (NT <= 128) {
+    if (NT <= 128 && !EXPERTS) {
         // Cut K while the slices of all tiles fit the device at once (two CTAs per SM keep enough copies in flight) and are
         // at least two blocks long.  Powers of two: clusters of other sizes do not fill the SM groups.
         while (p.ksplit < kMaxSplit && tiles * p.ksplit * 2 <= sms * G::PER_SM && p.kblocks >= 4 * p.ksplit) p.ksplit *= 2;
     }
     int grid = tiles * p.ksplit;
-    if (p.ksplit == 1 && G::NACC > 1 && grid > sms) grid = sms;     // persistent
+    if (EXPERTS) {
+        // at most one partly filled token tile per expert
+        const long long most = (long long)p.gtiles * (rows / NT + (rows < groups ? rows : groups));
+        grid = most < sms * G::PER_SM ? (int)most : sms * G::PER_SM;
+    } else if (p.ksplit == 1 && G::NACC > 1 && grid > sms) {
+        grid = sms;                                                 // persistent
+    }
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(grid);
     cfg.blockDim = dim3(kThreads);
@@ -370,24 +460,30 @@ int launch_gemm(const b200_linear& lin, const void* x, int x_rows, const Epi& ep
 }
 
 // ---------------------------------------------------------------- fp32 activations
+struct F32Params {
+    const bf16* w;
+    const float* x;
+    int n, npad, groups, pitch, x_pitch;      // rows of a group, as stored
+};
+
 // Few rows: one warp per output column, the rows in groups of 8.
-__global__ void __launch_bounds__(256) linear_f32_rows_kernel(const bf16* w, const float* x, int N, int pitch,
-                                                              const __grid_constant__ Epi epi) {
+__global__ void __launch_bounds__(256) linear_f32_rows_kernel(const F32Params p, const __grid_constant__ Epi epi) {
     pdl_wait();
     pdl_launch_dependents();
-    const int n = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (n >= N) return;
+    const int nr = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, g = nr / p.npad, r = nr - g * p.npad;
+    if (g >= p.groups || r >= p.n) return;
     ColumnOut<float> out;
-    out.init(epi, n);
-    const bf16* wr = w + (size_t)n * pitch;
+    out.init(epi, g * p.n + r);
+    const bf16* wr = p.w + (size_t)nr * p.pitch;
+    const float* x = p.x + (size_t)g * p.pitch;
     for (int m0 = 0; m0 < epi.M; m0 += 8) {
         float acc[8] = {};
-        for (int k = lane * 2; k < pitch; k += 64) {
+        for (int k = lane * 2; k < p.pitch; k += 64) {
             const float2 wv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(wr + k));
 #pragma unroll
             for (int i = 0; i < 8; i++)
                 if (m0 + i < epi.M) {
-                    const float2 xv = *reinterpret_cast<const float2*>(x + (size_t)(m0 + i) * pitch + k);
+                    const float2 xv = *reinterpret_cast<const float2*>(x + (size_t)(m0 + i) * p.x_pitch + k);
                     acc[i] = fmaf(wv.x, xv.x, acc[i]);
                     acc[i] = fmaf(wv.y, xv.y, acc[i]);
                 }
@@ -401,20 +497,21 @@ __global__ void __launch_bounds__(256) linear_f32_rows_kernel(const bf16* w, con
 }
 
 // Many rows: 64 columns x 64 rows per CTA, 4 x 4 per thread.
-__global__ void __launch_bounds__(256) linear_f32_tile_kernel(const bf16* w, const float* x, int N, int pitch,
-                                                              const __grid_constant__ Epi epi) {
+__global__ void __launch_bounds__(256) linear_f32_tile_kernel(const F32Params p, const __grid_constant__ Epi epi) {
     pdl_wait();
     pdl_launch_dependents();
     __shared__ float sw[16][68], sx[16][68];
-    const int n0 = blockIdx.x * 64, m0 = blockIdx.y * 64;
+    const int n0 = blockIdx.x * 64, m0 = blockIdx.y * 64, g = n0 / p.npad, c0 = n0 - g * p.npad;
+    if (c0 >= p.n) return;
     const int tn = threadIdx.x & 15, tm = threadIdx.x >> 4;
+    const float* x = p.x + (size_t)g * p.pitch;
     float acc[4][4] = {};
-    for (int k0 = 0; k0 < pitch; k0 += 16) {
+    for (int k0 = 0; k0 < p.pitch; k0 += 16) {
 #pragma unroll
         for (int i = 0; i < 4; i++) {
             const int e = threadIdx.x + 256 * i, r = e >> 4, k = e & 15;
-            sw[k][r] = n0 + r < N ? __bfloat162float(w[(size_t)(n0 + r) * pitch + k0 + k]) : 0.f;
-            sx[k][r] = m0 + r < epi.M ? x[(size_t)(m0 + r) * pitch + k0 + k] : 0.f;
+            sw[k][r] = c0 + r < p.n ? __bfloat162float(p.w[(size_t)(n0 + r) * p.pitch + k0 + k]) : 0.f;
+            sx[k][r] = m0 + r < epi.M ? x[(size_t)(m0 + r) * p.x_pitch + k0 + k] : 0.f;
         }
         __syncthreads();
 #pragma unroll
@@ -431,10 +528,10 @@ __global__ void __launch_bounds__(256) linear_f32_tile_kernel(const bf16* w, con
     }
 #pragma unroll
     for (int i = 0; i < 4; i++) {
-        const int n = n0 + tn + 16 * i;
-        if (n >= N) continue;
+        const int c = c0 + tn + 16 * i;
+        if (c >= p.n) continue;
         ColumnOut<float> out;
-        out.init(epi, n);
+        out.init(epi, g * p.n + c);
 #pragma unroll
         for (int j = 0; j < 4; j++)
             if (m0 + tm + 16 * j < epi.M) out.store(m0 + tm + 16 * j, acc[i][j]);
@@ -443,23 +540,38 @@ __global__ void __launch_bounds__(256) linear_f32_tile_kernel(const bf16* w, con
 
 }  // namespace
 
-int launch_linear(int act_type, const b200_linear& lin, const void* x, int x_rows, const Epi& epi, int* error, cudaStream_t st) {
+int launch_linear(int act_type, const b200_linear& lin, const void* x, int x_pitch, int x_rows, const Epi& epi, int* error, cudaStream_t st) {
     if (!lin.w || !x || lin.n < 1 || lin.pitch < 64 || lin.pitch % 64 != 0 || epi.M < 1 || x_rows < epi.M) return B200_EINVAL;
-    if (!aligned16(lin.w) || !aligned16(x)) return B200_EALIGN;
+    const int groups = lin.groups > 1 ? lin.groups : 1;
+    if (x_pitch == 0) x_pitch = groups * lin.pitch;
+    if (!aligned16(lin.w) || !aligned16(x) || x_pitch % 8 != 0) return B200_EALIGN;
     if (act_type == B200_ACT_F32) {
+        if (x_pitch < groups * lin.pitch || epi.gate.kind != 0) return B200_EINVAL;
+        const int npad = round_up(lin.n, kTileRows);
+        const F32Params p{static_cast<const bf16*>(lin.w), static_cast<const float*>(x), lin.n, npad, groups, lin.pitch, x_pitch};
         if (epi.M <= 16)
-            launch_kernel(linear_f32_rows_kernel, dim3((lin.n + 7) / 8), dim3(256), 0, st, static_cast<const bf16*>(lin.w),
-                          static_cast<const float*>(x), lin.n, lin.pitch, epi);
+            launch_kernel(linear_f32_rows_kernel, dim3(groups * npad / 8), dim3(256), 0, st, p, epi);
         else
-            launch_kernel(linear_f32_tile_kernel, dim3((lin.n + 63) / 64, (epi.M + 63) / 64), dim3(256), 0, st,
-                          static_cast<const bf16*>(lin.w), static_cast<const float*>(x), lin.n, lin.pitch, epi);
+            launch_kernel(linear_f32_tile_kernel, dim3(groups * npad / 64, (epi.M + 63) / 64), dim3(256), 0, st, p, epi);
         return check_launch();
     }
-    if (epi.M <= 16) return launch_gemm<16>(lin, x, x_rows, epi, error, st);
-    if (epi.M <= 32) return launch_gemm<32>(lin, x, x_rows, epi, error, st);
-    if (epi.M <= 64) return launch_gemm<64>(lin, x, x_rows, epi, error, st);
-    if (epi.M <= 128) return launch_gemm<128>(lin, x, x_rows, epi, error, st);
-    return launch_gemm<256>(lin, x, x_rows, epi, error, st);
+    const int M = epi.M, tiles = groups * ((lin.n + kTileRows - 1) / kTileRows);
+    if (M <= 16) return launch_gemm<16, false>(lin, x, x_pitch, x_rows, epi, M, nullptr, error, st);
+    if (M <= 32) return launch_gemm<32, false>(lin, x, x_pitch, x_rows, epi, M, nullptr, error, st);
+    // (few output columns: small token tiles, so that more SMs take part)
+    if (M <= 64 || tiles * ((M + 255) / 256) * 2 <= sm_count()) return launch_gemm<64, false>(lin, x, x_pitch, x_rows, epi, M, nullptr, error, st);
+    if (M <= 128) return launch_gemm<128, false>(lin, x, x_pitch, x_rows, epi, M, nullptr, error, st);
+    return launch_gemm<256, false>(lin, x, x_pitch, x_rows, epi, M, nullptr, error, st);
+}
+
+int launch_linear_experts(const b200_linear& lin, const void* x, int x_rows, int rows, const int* offsets, const Epi& epi, int* error, cudaStream_t st) {
+    if (!lin.w || !x || !offsets || lin.n < 1 || lin.pitch < 64 || lin.pitch % 64 != 0 || rows < 1 || x_rows < rows) return B200_EINVAL;
+    if (lin.groups < 1 || lin.groups > B200_HYBRID_MAX_EXPERTS) return B200_ELIMIT;
+    if (!aligned16(lin.w) || !aligned16(x)) return B200_EALIGN;
+    const int mean = rows / lin.groups;
+    if (mean <= 24) return launch_gemm<32, true>(lin, x, lin.pitch, x_rows, epi, rows, offsets, error, st);
+    if (mean <= 80) return launch_gemm<64, true>(lin, x, lin.pitch, x_rows, epi, rows, offsets, error, st);
+    return launch_gemm<128, true>(lin, x, lin.pitch, x_rows, epi, rows, offsets, error, st);
 }
 
 }  // namespace hybrid

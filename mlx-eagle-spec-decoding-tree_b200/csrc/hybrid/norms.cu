@@ -1,5 +1,6 @@
 // Element-wise and per-row steps of the hybrid decoders: embedding, RMS norm with the causal input convolution, RMS
-// norm alone (feed-forward input, final norm with row gather), the polynomial activation, stream injection.  All
+// norm alone (feed-forward input, final norm with row gather), a sublayer's normed output joined to the stream, the
+// polynomial and the gated activation, stream injection.  All
 // statistics and the residual stream are fp32; outputs that feed a product have the activation type.
 #include "hybrid.cuh"
 
@@ -36,24 +37,39 @@ template <int V> __device__ __forceinline__ void st(bf16* p, const Vec<V>& r) {
     }
 }
 
-__global__ void __launch_bounds__(kThreads) embed_kernel(const int* tokens, const bf16* table, int width, int vocab, float* x, float* emb) {
+struct EmbedParams {
+    const int* tokens;
+    const bf16* table;
+    float* x;
+    float* emb;                      // copy of the output, or null
+    void* out;                       // product input [M][pitch], or null
+    const int* pos;
+    int* tail_pos;                   // tree: positions of the tail rows (null: chain)
+    int width, vocab, pitch;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(kThreads) embed_kernel(const EmbedParams p) {
     pdl_launch_dependents();
     pdl_wait();
     constexpr int N = 4;                              // channels of a thread; all loads before the first store
     const int m = blockIdx.x, c0 = blockIdx.y * kThreads * N + threadIdx.x;
-    const int tok = min(max(tokens[m], 0), vocab - 1);
-    const bf16* src = table + (size_t)tok * width;
+    const int tok = min(max(p.tokens[m], 0), p.vocab - 1);
+    const bf16* src = p.table + (size_t)tok * p.width;
     bf16 v[N];
 #pragma unroll
-    for (int i = 0; i < N; i++) v[i] = c0 + i * kThreads < width ? src[c0 + i * kThreads] : __float2bfloat16_rn(0.f);
+    for (int i = 0; i < N; i++) v[i] = c0 + i * kThreads < p.width ? src[c0 + i * kThreads] : __float2bfloat16_rn(0.f);
 #pragma unroll
     for (int i = 0; i < N; i++) {
         const int c = c0 + i * kThreads;
-        if (c < width) {
-            x[(size_t)m * width + c] = __bfloat162float(v[i]);
-            if (emb != nullptr) emb[(size_t)m * width + c] = __bfloat162float(v[i]);
+        if (c < p.width) {
+            const float f = __bfloat162float(v[i]);
+            p.x[(size_t)m * p.width + c] = f;
+            if (p.emb != nullptr) p.emb[(size_t)m * p.width + c] = f;
+            if (p.out != nullptr) static_cast<T*>(p.out)[(size_t)m * p.pitch + c] = from_f32<T>(f);
         }
     }
+    if (p.tail_pos != nullptr && blockIdx.y == 0 && threadIdx.x == 0) p.tail_pos[m] = p.pos[m];
 }
 
 template <int V>
@@ -79,8 +95,6 @@ struct NormConvParams {
     float* pend;                     // [64][width] inputs of this pass's rows until they are committed
     void* out;                       // [M][pitch]
     const unsigned long long* mask;
-    const int* pos;
-    int* tail_pos;
     int M, width, pitch, write_off;
     float eps;
 };
@@ -119,7 +133,6 @@ __global__ void __launch_bounds__(kThreads) norm_conv_kernel(const NormConvParam
                     s_src[j] = p.state + (size_t)(j + have) * W;
                 }
             }
-            if (blockIdx.y == 0) p.tail_pos[self] = p.pos[r0];
         }
         __syncthreads();
     }
@@ -239,6 +252,73 @@ __global__ void __launch_bounds__(1024) polynorm_kernel(const T* z, T* out, int 
     }
 }
 
+// x += y / rms(y) * w (w null: x += mult * y), y the sum of `slots` rows; the new stream also goes to the product input.
+struct JoinParams {
+    const float* y;
+    const float* w;
+    const int* place;                // rows of y of every (row, slot), null: row * slots + slot
+    const float* add;
+    float* x;
+    void* out;
+    int slots, width, pitch;
+    float eps, mult;
+};
+
+template <typename T, int V>
+__global__ void __launch_bounds__(1024) join_kernel(const JoinParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    extern __shared__ __align__(16) float s_y[];      // the row's y
+    __shared__ float red[33];
+    __shared__ int s_row[B200_HYBRID_MAX_TOP];
+    const int m = blockIdx.x;
+    if (threadIdx.x < p.slots) s_row[threadIdx.x] = p.place != nullptr ? p.place[m * p.slots + threadIdx.x] : m * p.slots + threadIdx.x;
+    __syncthreads();
+    float ss = 0.f;
+#pragma unroll 2
+    for (int c = threadIdx.x * V; c < p.width; c += blockDim.x * V) {
+        Vec<V> t = ld<V>(p.y + (size_t)s_row[0] * p.width + c);
+        for (int s = 1; s < p.slots; s++) {
+            const Vec<V> u = ld<V>(p.y + (size_t)s_row[s] * p.width + c);
+#pragma unroll
+            for (int e = 0; e < V; e++) t.v[e] += u.v[e];
+        }
+#pragma unroll
+        for (int e = 0; e < V; e++) ss = fmaf(t.v[e], t.v[e], ss);
+        st<V>(s_y + c, t);
+    }
+    float f = p.mult;
+    if (p.w != nullptr) f = rsqrtf(block_sum(ss, red) / (float)p.width + p.eps);
+    float* x = p.x + (size_t)m * p.width;
+    T* o = static_cast<T*>(p.out) + (size_t)m * p.pitch;
+#pragma unroll 2
+    for (int c = threadIdx.x * V; c < p.width; c += blockDim.x * V) {      // (each thread its own channels)
+        const Vec<V> t = ld<V>(s_y + c);
+        Vec<V> g, r = ld<V>(x + c);
+        if (p.w != nullptr) g = ld<V>(p.w + c);
+#pragma unroll
+        for (int e = 0; e < V; e++) r.v[e] += p.w != nullptr ? t.v[e] * f * g.v[e] : t.v[e] * f;
+        if (p.add != nullptr) {
+            const Vec<V> a = ld<V>(p.add + (size_t)m * p.width + c);
+#pragma unroll
+            for (int e = 0; e < V; e++) r.v[e] += a.v[e];
+        }
+        st<V>(x + c, r);
+        st<V>(o + c, r);
+    }
+}
+
+// Columns alternating gate and up -> the activation (fp32 products, whose epilogue does not pair columns).
+__global__ void __launch_bounds__(kThreads) gated_kernel(const float* z, int z_pitch, float* out, int pitch, int ff, const float* bias, Gating gate) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int c = blockIdx.x * kThreads + threadIdx.x, m = blockIdx.y;
+    if (c >= ff) return;
+    float g = z[(size_t)m * z_pitch + 2 * c], u = z[(size_t)m * z_pitch + 2 * c + 1];
+    if (bias != nullptr) { g += bias[2 * c]; u += bias[2 * c + 1]; }
+    out[(size_t)m * pitch + c] = gated_f(gate, g, u);
+}
+
 __global__ void add_kernel(float* x, const float* y, size_t n) {
     pdl_launch_dependents();
     pdl_wait();
@@ -249,8 +329,13 @@ __global__ void add_kernel(float* x, const float* y, size_t n) {
 }  // namespace
 
 int launch_embed(const b200_hybrid_model& m, const b200_hybrid_pass& p, cudaStream_t st) {
-    launch_kernel(embed_kernel, dim3(p.M, (m.width + 4 * kThreads - 1) / (4 * kThreads)), dim3(kThreads), 0, st, p.tokens, static_cast<const bf16*>(m.embed), m.width, m.vocab, m.x,
-                  m.injects ? m.emb : static_cast<float*>(nullptr));
+    EmbedParams q{};
+    q.tokens = p.tokens; q.table = static_cast<const bf16*>(m.embed); q.x = m.x; q.emb = m.injects ? m.emb : nullptr;
+    q.out = m.norm_out ? m.hb : nullptr; q.pos = p.pos; q.tail_pos = p.tree ? p.tail_pos + p.write_off : nullptr;
+    q.width = m.width; q.vocab = m.vocab; q.pitch = round_up(m.width, 64);
+    const dim3 grid(p.M, (m.width + 4 * kThreads - 1) / (4 * kThreads));
+    if (m.act_type == B200_ACT_F32) launch_kernel(embed_kernel<float>, grid, dim3(kThreads), 0, st, q);
+    else launch_kernel(embed_kernel<bf16>, grid, dim3(kThreads), 0, st, q);
     return check_launch();
 }
 
@@ -305,6 +390,16 @@ int launch_polynorm_t(const b200_hybrid_model& m, const b200_hybrid_layer& l, in
     return check_launch();
 }
 
+template <typename T>
+int launch_join_t(const JoinParams& p, int rows, cudaStream_t st) {
+    const size_t smem = (size_t)p.width * 4;
+    if (smem > 160 * 1024) return B200_ELIMIT;
+    auto k = p.width % 4 == 0 ? join_kernel<T, 4> : join_kernel<T, 1>;
+    if (smem > 40 * 1024 && cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return check_launch();
+    launch_kernel(k, dim3(rows), dim3(row_threads(rows, p.width % 4 == 0 ? p.width / 4 : p.width)), smem, st, p);
+    return check_launch();
+}
+
 }  // namespace
 
 int launch_norm_conv(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_run& r, const b200_hybrid_pass& p,
@@ -313,7 +408,7 @@ int launch_norm_conv(const b200_hybrid_model& m, const b200_hybrid_layer& l, con
     q.x = m.x; q.w = l.norm1; q.conv = l.conv;
     q.state = reinterpret_cast<const float*>(static_cast<const char*>(p.cache) + r.conv_off);
     q.pend = reinterpret_cast<float*>(static_cast<char*>(m.pending) + r.pend_h);
-    q.out = m.hb; q.mask = p.mask; q.pos = p.pos; q.tail_pos = p.tail_pos;
+    q.out = m.hb; q.mask = p.mask;
     q.M = p.M; q.width = m.width; q.pitch = round_up(m.width, 64); q.write_off = p.write_off;
     q.eps = m.eps;
     return m.act_type == B200_ACT_F32 ? launch_norm_conv_t<float, 1>(q, l.taps, p.tree, st) : launch_norm_conv_t<bf16, 1>(q, l.taps, p.tree, st);
@@ -325,6 +420,21 @@ int launch_norm(const b200_hybrid_model& m, const float* w, const b200_hybrid_pa
 
 int launch_polynorm(const b200_hybrid_model& m, const b200_hybrid_layer& l, int rows, cudaStream_t st) {
     return m.act_type == B200_ACT_F32 ? launch_polynorm_t<float>(m, l, rows, st) : launch_polynorm_t<bf16>(m, l, rows, st);
+}
+
+int launch_join(const b200_hybrid_model& m, const float* w, int rows, int slots, const int* place, const float* x_add, cudaStream_t st) {
+    if (slots < 1 || slots > B200_HYBRID_MAX_TOP) return B200_ELIMIT;
+    JoinParams p{};
+    p.y = m.y; p.w = w; p.place = place; p.add = x_add; p.x = m.x; p.out = m.hb; p.slots = slots; p.width = m.width;
+    p.pitch = round_up(m.width, 64); p.eps = m.eps; p.mult = m.residual_mult;
+    return m.act_type == B200_ACT_F32 ? launch_join_t<float>(p, rows, st) : launch_join_t<bf16>(p, rows, st);
+}
+
+int launch_gated(const b200_hybrid_model& m, const b200_hybrid_layer& l, int rows, cudaStream_t st) {
+    if (m.act_type != B200_ACT_F32) return B200_EINVAL;
+    launch_kernel(gated_kernel, dim3((l.ff + kThreads - 1) / kThreads, rows), dim3(kThreads), 0, st, static_cast<const float*>(m.zb),
+                  round_up(2 * l.ff, 64), static_cast<float*>(m.zab), round_up(l.ff, 64), l.ff, l.up_bias, gating_of(l));
+    return check_launch();
 }
 
 int launch_add(float* x, const float* y, size_t n, cudaStream_t st) {

@@ -9,9 +9,8 @@
 //   tree_kernel    tree passes: nothing may change the state yet.  Row m's output is written out along its path:
 //                  o = S_0^T (q prod f) + sum over the path's rows a of (q . (1 - f_a) prod of the later f) v_a.
 //   commit_kernel  advances convolution inputs, states and K/V rows over accepted rows, for every layer run at once.
-//   head_norm      per-head RMS norm of the outputs with the head weight, to the activation type.
-#include "hybrid.cuh"
-#include "../pipeline.cuh"
+//   head_norm      per-head RMS norm of the outputs with the head weight (times a gate), to the activation type.
+#include "scan.cuh"
 
 namespace b200 {
 namespace hybrid {
@@ -21,22 +20,6 @@ constexpr int kWarps = 8;
 constexpr int kLaneCols = 4;         // state columns of a warp of the scan
 constexpr int kMaxDim = 256;
 
-// Two fp32 values in one register pair: packed multiply-adds, each half rounded as a single one.
-__device__ __forceinline__ unsigned long long pack2(float a, float b) {
-    unsigned long long r;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-    return r;
-}
-__device__ __forceinline__ float2 unpack2(unsigned long long v) {
-    float2 r;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
-    return r;
-}
-__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
-    unsigned long long r;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-    return r;
-}
 constexpr unsigned long long kMinusOne2 = 0xbf800000bf800000ull;
 
 // Sum of v[i] over the warp's lanes, for 32 values at once: lane i gets the total of v[i].
@@ -63,16 +46,6 @@ template <int RPL> __device__ __forceinline__ void ld_pairs(unsigned long long (
         const uint32_t u = *reinterpret_cast<const uint32_t*>(p + 2 * i);
         r[i] = pack2(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u));
     }
-}
-
-// One row of `n` elements to shared memory by a warp: 16-byte asynchronous copies where the row allows them.
-template <typename E>
-__device__ __forceinline__ void fetch_row(E* dst, const E* src, int n, bool wide, int lane) {
-    constexpr int VE = 16 / (int)sizeof(E);
-    if (wide)
-        for (int c = lane * VE; c < n; c += 32 * VE) cp_async16(smem_u32(dst + c), src + c);
-    else
-        for (int c = lane; c < n; c += 32) dst[c] = src[c];
 }
 
 template <typename T, int RPL>           // state rows of a lane
@@ -237,7 +210,7 @@ __global__ void __launch_bounds__(128) tree_kernel(const T* q, const float* pend
 }
 
 template <typename T>
-__global__ void __launch_bounds__(128) head_norm_kernel(const float* o, const float* w, T* out, int M, int H,
+__global__ void __launch_bounds__(128) head_norm_kernel(const float* o, const float* w, const T* gate, T* out, int M, int H,
                                                         int dv, int pitch, float eps) {
     pdl_launch_dependents();
     pdl_wait();
@@ -249,6 +222,11 @@ __global__ void __launch_bounds__(128) head_norm_kernel(const float* o, const fl
     for (int c = lane; c < dv; c += 32) { const float x = row[c]; ss = fmaf(x, x, ss); }
     const float rstd = rsqrtf(warp_sum(ss) / (float)dv + eps);
     T* dst = out + (size_t)m * pitch + (size_t)h * dv;
+    if (gate != nullptr) {
+        const T* g = gate + (size_t)unit * dv;
+        for (int c = lane; c < dv; c += 32) dst[c] = from_f32<T>(row[c] * rstd * w[c] * to_f32<T>(g[c]));
+        return;
+    }
     for (int c = lane; c < dv; c += 32) dst[c] = from_f32<T>(row[c] * rstd * w[c]);
 }
 
@@ -312,10 +290,11 @@ __global__ void __launch_bounds__(256) commit_kernel(const CommitParams p) {
             state[e] = s;
         }
     }
-    if (p.compact && l.mixer == B200_MIXER_ATTENTION) {
+    if (p.compact && (l.mixer == B200_MIXER_ATTENTION || l.mixer == B200_MIXER_LATENT)) {
         const int P = p.prefix[0];
-        const int ke = l.maps * round_up(l.dim, 16), ve = round_up(l.vdim, 16), per = ke + ve;
-        for (int e = first; e < l.kv_heads * per; e += step) {
+        const bool latent = l.mixer == B200_MIXER_LATENT;           // one row per token for all heads, no values of their own
+        const int ke = latent ? latent_pitch(l) : l.maps * round_up(l.dim, 16), ve = latent ? 0 : round_up(l.vdim, 16), per = ke + ve;
+        for (int e = first; e < (latent ? 1 : l.kv_heads) * per; e += step) {
             const int g = e / per, x = e - g * per;
             T* base = x < ke ? reinterpret_cast<T*>(p.cache + r.k_off) + (size_t)g * p.cap * ke + x
                              : reinterpret_cast<T*>(p.cache + r.v_off) + (size_t)g * p.cap * ve + (x - ke);
@@ -352,13 +331,22 @@ int recurrence(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b20
     } else {
         rc = launch_scan<T>(m, l, state, p.M, st);
     }
-    if (rc != B200_OK) return rc;
-    launch_kernel(head_norm_kernel<T>, dim3((p.M * l.heads + 3) / 4), dim3(128), 0, st, static_cast<const float*>(m.o32), l.head_norm,
-                  static_cast<T*>(m.ab), p.M, l.heads, l.vdim, round_up(l.heads * l.vdim, 64), m.eps);
-    return check_launch();
+    return rc != B200_OK ? rc : launch_head_norm(m, l, p.M, nullptr, st);
+}
+
+template <typename T>
+void launch_head_norm_t(const b200_hybrid_model& m, const b200_hybrid_layer& l, int rows, const void* gate, cudaStream_t st) {
+    launch_kernel(head_norm_kernel<T>, dim3((rows * l.heads + 3) / 4), dim3(128), 0, st, static_cast<const float*>(m.o32), l.head_norm,
+                  static_cast<const T*>(gate), static_cast<T*>(m.ab), rows, l.heads, l.vdim, round_up(l.heads * l.vdim, 64), m.eps);
 }
 
 }  // namespace
+
+int launch_head_norm(const b200_hybrid_model& m, const b200_hybrid_layer& l, int rows, const void* gate, cudaStream_t st) {
+    if (m.act_type == B200_ACT_F32) launch_head_norm_t<float>(m, l, rows, gate, st);
+    else launch_head_norm_t<bf16>(m, l, rows, gate, st);
+    return check_launch();
+}
 
 int launch_recurrence(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_run& r, const b200_hybrid_pass& p,
                       cudaStream_t st) {

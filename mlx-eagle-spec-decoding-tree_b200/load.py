@@ -35,7 +35,7 @@ import numpy as np
 import torch
 
 from . import _lib
-from .hybrid import HybridArgs, HybridModel, preset_config
+from .hybrid import DESIGNS, HybridArgs, HybridModel, preset_config
 from .llama import Model, ModelArgs, QLinear, shape_preset
 
 _DTYPES = {"U32": (np.uint32, 4), "I32": (np.int32, 4), "F16": (np.float16, 2), "F32": (np.float32, 4),
@@ -211,7 +211,7 @@ def _load_quantised(model_path: str, config: dict, device, dtype: str) -> Model:
 
 # name in config.json -> (builder, kernel library, does it run in fp32)
 MODEL_TYPES = {"llama": (_load_quantised, "eagle", False), "qwen2": (_load_quantised, "eagle", False)}
-ARCHITECTURES = {"Zaverax": (_load_hybrid, "hybrid", True)}
+ARCHITECTURES = {name: (_load_hybrid, "hybrid", True) for name in DESIGNS}
 
 
 def load(path: str, device, tokenizer_config: Optional[dict] = None, model_config: Optional[dict] = None, dtype: str = "bfloat16"):

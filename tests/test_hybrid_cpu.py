@@ -24,12 +24,20 @@ def test_header_symbols_are_exported(be):
         assert hasattr(be._lib.hybrid(), n), n
 
 
-def test_struct_mirrors(be):
+def test_struct_mirrors(be, tmp_path):
+    """Sizes and field offsets of the ctypes mirrors against the header, as a C compiler lays it out."""
     L = be._lib
-    assert ctypes.sizeof(L.Linear) == 24
-    assert ctypes.sizeof(L.HybridLayer) == 10 * 4 + 3 * 4 + 4 * 4 + 4 + 6 * 8 + 4 * 24
-    assert ctypes.sizeof(L.HybridRun) == 8 + 7 * 8
-    assert ctypes.sizeof(L.HybridPass) == 8 * 4 + 11 * 8
+    mirrors = {"b200_linear": L.Linear, "b200_hybrid_layer": L.HybridLayer, "b200_hybrid_run": L.HybridRun, "b200_hybrid_model": L.HybridModelDesc,
+               "b200_hybrid_pass": L.HybridPass}
+    fields = [(s, c, f[0]) for s, c in mirrors.items() for f in c._fields_]
+    c_name = {"in_": "in", "lambda_": "lambda"}
+    prog = "#include <stdio.h>\n#include <stddef.h>\n#include \"b200_hybrid.h\"\nint main(void) {\n"
+    prog += "".join(f'printf("%zu\\n", sizeof({s}));\n' for s in mirrors)
+    prog += "".join(f'printf("%zu\\n", offsetof({s}, {c_name.get(f, f)}));\n' for s, _, f in fields) + "return 0; }\n"
+    (tmp_path / "sizes.c").write_text(prog)
+    subprocess.run(["gcc", "-I", os.path.join(ROOT, "include"), str(tmp_path / "sizes.c"), "-o", str(tmp_path / "sizes")], check=True, timeout=120)
+    got = [int(x) for x in subprocess.run([str(tmp_path / "sizes")], capture_output=True, text=True, check=True, timeout=60).stdout.split()]
+    assert got == [ctypes.sizeof(c) for c in mirrors.values()] + [getattr(c, f).offset for _, c, f in fields]
 
 
 def test_bad_arguments_are_refused_before_any_launch(be):
