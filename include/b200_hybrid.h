@@ -133,6 +133,7 @@ typedef struct b200_hybrid_model {
     float* q32;                         /* delta: unit queries and keys [max_rows][kv_heads*dim]                     */
     float* k32;
     float* beta;                        /* delta: [max_rows][heads]                                                  */
+    float* chunk;                       /* delta: floats of b200_hybrid_chunk_floats                                 */
     float* lat32;                       /* latent: rotated query parts | latent | rotated key part, before norm and rotation */
     void* qn;                           /* latent: unrotated queries [max_rows][heads][dim64]                        */
     void* ob;                           /* latent: attention output over the latent [max_rows][heads][kv_rank64]     */
@@ -171,6 +172,9 @@ typedef struct b200_hybrid_pass {
 
 /* Bytes of attention partials a pass of `rows` tree rows (or fp32 / short chain rows) needs at most. */
 size_t b200_hybrid_attention_workspace_bytes(const b200_hybrid_model* model, int rows);
+
+/* Floats of `chunk`: vectors and coefficients of a delta layer's prompt rows, 8 tokens at a time. */
+size_t b200_hybrid_chunk_floats(int max_rows, int heads, int dim);
 
 /* Ints of `route`: expert and position of every (row, choice), the choices' scores, first place of every expert. */
 size_t b200_hybrid_route_ints(int max_rows, int top, int experts);

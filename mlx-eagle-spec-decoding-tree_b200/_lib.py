@@ -59,6 +59,8 @@ def hybrid() -> ctypes.CDLL:
         l.b200_hybrid_set_pdl.argtypes = [i32]
         l.b200_hybrid_attention_workspace_bytes.restype = sz
         l.b200_hybrid_attention_workspace_bytes.argtypes = [mp, i32]
+        l.b200_hybrid_chunk_floats.restype = sz
+        l.b200_hybrid_chunk_floats.argtypes = [i32, i32, i32]
         l.b200_hybrid_route_ints.restype = sz
         l.b200_hybrid_route_ints.argtypes = [i32, i32, i32]
         l.b200_hybrid_forward.restype = i32
@@ -235,7 +237,7 @@ class HybridModelDesc(ctypes.Structure):
                 + [("layers", ctypes.POINTER(HybridLayer)), ("runs", ctypes.POINTER(HybridRun))]
                 + [(n, ctypes.c_void_p) for n in ("dev_layers", "dev_runs")] + [("head", Linear)]
                 + [(n, ctypes.c_void_p) for n in ("x", "emb", "hb", "qb", "gb", "vb", "gf", "o32", "ab", "zb", "zab",
-                                                  "y", "cb", "lowb", "q32", "k32", "beta", "lat32", "qn", "ob", "kx", "vx",
+                                                  "y", "cb", "lowb", "q32", "k32", "beta", "chunk", "lat32", "qn", "ob", "kx", "vx",
                                                   "zr", "route", "xg")]
                 + [(n, ctypes.c_int) for n in ("x_rows", "route_top", "route_experts", "reserved")]
                 + [(n, ctypes.c_void_p) for n in ("pending", "attn_part")]

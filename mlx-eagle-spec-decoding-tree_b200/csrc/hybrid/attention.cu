@@ -12,18 +12,16 @@
 // mma.sync with the key/value blocks double-buffered by cp.async; both maps share the value block.  The softmax weights
 // enter the value product as a pair of bf16 terms (value + remainder), which keeps them at fp32-like precision.
 //
-// Latent attention (one low-rank latent and one rotated key part per token, shared by all heads) uses both: few rows walk the
-// latent itself, with queries brought into its space and the key row's first columns as values (SHARED); prompts walk keys
-// and values written out per head, the rotated part taken from the cache (LATENT).
-#include "hybrid.cuh"
-#include "../pipeline.cuh"
+// Latent attention (one low-rank latent and one rotated key part per token, shared by all heads) uses both: fp32 rows walk the
+// latent itself, with queries brought into its space and the key row's first columns as values (SHARED; bf16: latent.cu);
+// prompts walk keys and values written out per head, the rotated part taken from the cache (LATENT).
+#include "mma.cuh"
 
 namespace b200 {
 namespace hybrid {
 namespace {
 
 constexpr int kKeys = 64;                // keys of a block
-constexpr float kLog2e = 1.4426950408889634f;
 constexpr int kMaxSplits = 32;
 constexpr int kRowThreads = 128;
 
@@ -260,23 +258,6 @@ __global__ void __launch_bounds__(kRowThreads) attention_merge_kernel(const Attn
 
 // ---------------------------------------------------------------- prompts
 constexpr int kQRows = 64;
-
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile(
-        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
-        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<const uint32_t*>(&v);
-}
 
 template <int VT, int MAPS, bool LATENT> // 16-column value tiles, maps per head
 __global__ void __launch_bounds__(128) attention_prompt_kernel(const AttnParams p) {
@@ -577,7 +558,11 @@ size_t attention_part_bytes(const b200_hybrid_model& m, int rows) {
         const b200_hybrid_layer& l = m.layers[i];
         if (l.mixer != B200_MIXER_ATTENTION && l.mixer != B200_MIXER_LATENT) continue;
         const size_t r = rows > 592 ? rows : 592;        // rows * splits never exceeds it (pick_splits)
-        const size_t b = r * l.heads * l.maps * (round_up(l.mixer == B200_MIXER_LATENT ? l.kv_rank : l.vdim, 16) + 2) * 4;
+        size_t b = r * l.heads * l.maps * (round_up(l.vdim, 16) + 2) * 4;
+        if (l.mixer == B200_MIXER_LATENT) {
+            const size_t vectors = r * l.heads, packed = latent_attention_parts(rows, l.heads);
+            b = (vectors > packed ? vectors : packed) * (round_up(l.kv_rank, 16) + 2) * 4;
+        }
         most = b > most ? b : most;
     }
     return most;
@@ -598,6 +583,7 @@ int launch_attention(const b200_hybrid_model& m, const b200_hybrid_layer& l, con
             p.q_pitch = l.heads * p.dp; p.out = m.ab; p.out_pitch = round_up(l.heads * l.vdim, 64); p.out_head = l.vdim;
             return launch_prompt_any<1, true>(p, st);
         }
+        if (m.act_type == B200_ACT_BF16 && cp <= kLatentColumns) return launch_latent_attention(m, l, r, ps, st);
         p.G = 1; p.dim = p.dp = cp + rp; p.vdim = l.kv_rank; p.vp = cp; p.kc = cache + r.k_off; p.cap = ps.cache_rows;
         p.q_pitch = l.heads * p.dp; p.out = m.ob; p.out_head = l.value.pitch; p.out_pitch = l.heads * l.value.pitch;
         return launch_latent_rows(m, l, p, ps.max_keys, st);

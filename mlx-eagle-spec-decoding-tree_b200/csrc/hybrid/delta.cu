@@ -4,12 +4,19 @@
 // fp32, the state [heads][vdim][dim] is carried in the request's cache, as are the convolutions' last inputs.
 //
 //   conv_kernel    convolution, silu and unit norm: a warp per head of q, k or v and block of rows.
-//   scan_kernel    CTA = (head, 32 state columns); 8 lanes share a column and hold its rows in registers (packed pairs), so the
-//                  read-out of k before the write takes three shuffles; tokens come in blocks through shared memory and the
-//                  lanes' parts of the outputs are added for 8 tokens at once.  Three forms:
+//   scan_kernel    token by token.  CTA = (head, 32 state columns); 8 lanes share a column and hold its rows in registers (packed
+//                  pairs), so the read-out of k before the write takes three shuffles; tokens come in blocks through shared
+//                  memory and the lanes' parts of the outputs are added for 8 tokens at once.  Three forms:
 //                    chain   the pass's rows in order; the new state and convolution inputs are written back;
 //                    tree    a CTA per row replays the row's path from the state, nothing is written back;
 //                    commit  pending rows are replayed and written back, no output.
+//   conv_chunk_kernel, chunk_scan_kernel
+//                  prompts: 8 tokens at a time.  With P_j the product of the chunk's decays up to token j and P_ij that of the
+//                  tokens after i up to j (products of decays only, nothing is divided),
+//                      u_j = beta_j (v_j - S^T (P_j k_j) - sum_{i<j} (k_j . P_ij k_i) u_i),
+//                      o_j = S^T (P_j q_j) + sum_{i<=j} (q_j . P_ij k_i) u_i,      S <- P_7 S + sum_i (P_i7 k_i) u_i^T
+//                  with S the state before the chunk: the read-outs of all 8 tokens are independent of each other.  The vectors
+//                  and the 8 x 8 coefficients do not depend on the column and come out of the convolution kernel.
 #include "scan.cuh"
 
 namespace b200 {
@@ -139,6 +146,166 @@ __global__ void __launch_bounds__(kThreads) conv_kernel(const ConvParams p) {
     }
 }
 
+// ---------------------------------------------------------------- 8 tokens at a time
+constexpr int kChunk = 8;
+
+// Sum of v[i] over the warp's lanes, for 32 values at once: lane i gets the total of v[i].
+__device__ __forceinline__ float transpose_sum32(float (&v)[32], int lane) {
+#pragma unroll
+    for (int s = 16; s > 0; s >>= 1)
+#pragma unroll
+        for (int i = 0; i < s; i++) {
+            const bool up = (lane & s) != 0;
+            const float keep = up ? v[i + s] : v[i], send = up ? v[i] : v[i + s];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, send, s);
+        }
+    return v[0];
+}
+
+struct ChunkParams {
+    ConvParams c;            // (q, k unused)
+    const float* g;          // [M][H * d]
+    float* kt;               // [M][H * d]: P_j k_j
+    float* qt;               // P_j q_j
+    float* kh;               // P_j7 k_j
+    float* decay;            // [chunks][H * d]: P_7
+    float* coef;             // [chunks][H][2][8][8]: k_j . P_ij k_i (i < j), q_j . P_ij k_i (i <= j), zeros elsewhere
+};
+
+// silu(convolution) of 8 rows from r0 on, the lane's 4 channels from c on (n of them in the head).
+template <typename T, int TAPS>
+__device__ __forceinline__ void conv_rows(const ConvParams& p, int r0, int rows, int c, bool in_head, float (&y)[kChunk][4]) {
+    constexpr int X = kChunk + TAPS - 1;
+    const T* in = static_cast<const T*>(p.in);
+    const T* state = static_cast<const T*>(p.state);
+    float x[X][4], w[TAPS][4];
+#pragma unroll
+    for (int i = 0; i < X; i++) {
+        const int row = r0 + i - (TAPS - 1);
+#pragma unroll
+        for (int e = 0; e < 4; e++) x[i][e] = 0.f;
+        if (in_head && row < r0 + rows) ld_vec<T, 4>(x[i], (row >= 0 ? in + (size_t)row * p.pitch : state + (size_t)(row + TAPS - 1) * p.pitch) + c);
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS; j++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) w[j][e] = in_head ? p.w[(size_t)j * p.channels + c + e] : 0.f;
+#pragma unroll
+    for (int r = 0; r < kChunk; r++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            float z = 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) z = fmaf(w[j][e], x[r + j][e], z);
+            y[r][e] = z * sigmoid_f(z);
+        }
+}
+
+// Warp = (chunk, key head) or (chunk, value head); heads of at most 128 channels, multiples of 4.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) conv_chunk_kernel(const ChunkParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const ConvParams& cp = p.c;
+    const int lane = threadIdx.x & 31, unit = blockIdx.x * 4 + (threadIdx.x >> 5), chunk = blockIdx.y, r0 = chunk * kChunk;
+    const int rows = min(kChunk, cp.M - r0), c = lane * 4, d = cp.d, G = cp.G, H = cp.H;
+    if (unit >= G + H) return;
+    if (unit >= G) {
+        const int h = unit - G;
+        const bool in = c < cp.dv;
+        float y[kChunk][4];
+        conv_rows<T, TAPS>(cp, r0, rows, 2 * G * d + h * cp.dv + c, in, y);
+#pragma unroll
+        for (int r = 0; r < kChunk; r++) {
+            if (!in || r >= rows) continue;
+            T* dst = static_cast<T*>(cp.v) + ((size_t)(r0 + r) * H + h) * cp.dv + c;
+            if constexpr (sizeof(T) == 4) {
+                *reinterpret_cast<float4*>(dst) = make_float4(y[r][0], y[r][1], y[r][2], y[r][3]);
+            } else {
+                const __nv_bfloat162 a = __floats2bfloat162_rn(y[r][0], y[r][1]), b = __floats2bfloat162_rn(y[r][2], y[r][3]);
+                *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+            }
+        }
+        return;
+    }
+    const bool in = c < d;
+    float q[kChunk][4], k[kChunk][4];
+    conv_rows<T, TAPS>(cp, r0, rows, unit * d + c, in, q);
+    conv_rows<T, TAPS>(cp, r0, rows, (G + unit) * d + c, in, k);
+    const float scale = rsqrtf((float)d);
+#pragma unroll
+    for (int r = 0; r < kChunk; r++) {
+        float sq = 0.f, sk = 0.f;
+#pragma unroll
+        for (int e = 0; e < 4; e++) { sq = fmaf(q[r][e], q[r][e], sq); sk = fmaf(k[r][e], k[r][e], sk); }
+        const float fq = rsqrtf(warp_sum(sq) + 1e-6f) * scale, fk = rsqrtf(warp_sum(sk) + 1e-6f);
+#pragma unroll
+        for (int e = 0; e < 4; e++) { q[r][e] *= fq; k[r][e] *= fk; }
+    }
+    // (rows past the pass are zero: zero inputs, or a head's zero channels)
+#pragma unroll
+    for (int r = 0; r < kChunk; r++)
+#pragma unroll
+        for (int e = 0; e < 4; e++)
+            if (r >= rows) q[r][e] = k[r][e] = 0.f;
+    const int R = H / G;
+    for (int h = unit * R; h < (unit + 1) * R; h++) {
+        float g[kChunk][4];
+#pragma unroll
+        for (int r = 0; r < kChunk; r++) {
+            float4 x = make_float4(1.f, 1.f, 1.f, 1.f);
+            if (in && r < rows) x = *reinterpret_cast<const float4*>(p.g + ((size_t)(r0 + r) * H + h) * d + c);
+            g[r][0] = x.x; g[r][1] = x.y; g[r][2] = x.z; g[r][3] = x.w;
+        }
+        float P[4] = {1.f, 1.f, 1.f, 1.f};
+#pragma unroll
+        for (int r = 0; r < kChunk; r++) {
+#pragma unroll
+            for (int e = 0; e < 4; e++) P[e] *= g[r][e];
+            if (in && r < rows) {
+                const size_t at = ((size_t)(r0 + r) * H + h) * d + c;
+                *reinterpret_cast<float4*>(p.kt + at) = make_float4(P[0] * k[r][0], P[1] * k[r][1], P[2] * k[r][2], P[3] * k[r][3]);
+                *reinterpret_cast<float4*>(p.qt + at) = make_float4(P[0] * q[r][0], P[1] * q[r][1], P[2] * q[r][2], P[3] * q[r][3]);
+            }
+        }
+        if (in) *reinterpret_cast<float4*>(p.decay + ((size_t)chunk * H + h) * d + c) = make_float4(P[0], P[1], P[2], P[3]);
+        float* coef = p.coef + ((size_t)chunk * H + h) * 2 * kChunk * kChunk;
+        *reinterpret_cast<float4*>(coef + lane * 4) = make_float4(0.f, 0.f, 0.f, 0.f);
+        __syncwarp();
+        // for every i: k_j . P_ij k_i for j > i, then q_j . P_ij k_i for j >= i; 64 sums in all, 32 at a time
+        float v[32];
+#pragma unroll
+        for (int i = 0, n = 0; i < kChunk; i++) {
+            float qd[kChunk], w[4];
+#pragma unroll
+            for (int e = 0; e < 4; e++) w[e] = k[i][e];
+            auto put = [&](float x) {
+                v[n & 31] = x;
+                n++;
+                if ((n & 31) == 0) {
+                    const float total = transpose_sum32(v, lane);
+                    int at = n - 32 + lane, ii = 0;
+                    while (at >= 15 - 2 * ii) { at -= 15 - 2 * ii; ii++; }
+                    const bool first = at < 7 - ii;
+                    const int jj = first ? ii + 1 + at : ii + at - (7 - ii);
+                    coef[(first ? 0 : kChunk * kChunk) + jj * kChunk + ii] = total;
+                }
+            };
+#pragma unroll
+            for (int j = i; j < kChunk; j++) {
+                if (j > i)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) w[e] *= g[j][e];
+                qd[j] = w[0] * q[j][0] + w[1] * q[j][1] + w[2] * q[j][2] + w[3] * q[j][3];
+                if (j > i) put(w[0] * k[j][0] + w[1] * k[j][1] + w[2] * k[j][2] + w[3] * k[j][3]);
+            }
+#pragma unroll
+            for (int j = i; j < kChunk; j++) put(qd[j]);
+            if (in && i < rows) *reinterpret_cast<float4*>(p.kh + ((size_t)(r0 + i) * H + h) * d + c) = make_float4(w[0], w[1], w[2], w[3]);
+        }
+    }
+}
+
 struct ScanParams {
     const float* q;          // [M][G * d]
     const float* k;          // chain: [M][G * d]; tree, commit: pending rows
@@ -170,6 +337,192 @@ __device__ __forceinline__ float transpose_sum8(float (&v)[8], int lane) {
             v[i] = keep + __shfl_xor_sync(0xffffffffu, send, s);
         }
     return v[0];
+}
+
+// The convolutions' last inputs after n rows, channels over all CTAs of the grid.
+template <typename T, typename RowOf>
+__device__ __forceinline__ void roll_inputs(const ScanParams& p, int n, RowOf row_of) {
+    const int prev = p.taps - 1, first = (blockIdx.y * gridDim.x + blockIdx.x) * blockDim.x + threadIdx.x;
+    const T* in = static_cast<const T*>(p.in);
+    T* cs = static_cast<T*>(p.conv_state);
+    if (prev == 0) return;
+    for (int c = first; c < p.channels; c += gridDim.x * gridDim.y * blockDim.x) {
+        T nv[B200_HYBRID_MAX_TAPS];
+#pragma unroll
+        for (int e = 0; e < B200_HYBRID_MAX_TAPS; e++)
+            if (e < prev) {
+                const int i = n - prev + e;
+                nv[e] = i >= 0 ? in[(size_t)row_of(i) * p.pitch + c] : cs[(size_t)(i + prev) * p.pitch + c];
+            }
+#pragma unroll
+        for (int e = 0; e < B200_HYBRID_MAX_TAPS; e++)
+            if (e < prev) cs[(size_t)e * p.pitch + c] = nv[e];
+    }
+}
+
+struct ChunkScanParams {
+    ScanParams s;
+    const float* kt;
+    const float* qt;
+    const float* kh;
+    const float* decay;
+    const float* coef;
+};
+
+// CTA = (head, 32 state columns), warp = 4 columns: 16 lanes share 2 columns and hold their rows.
+//
+// The read-outs of 4 tokens, of k and of q, for 2 columns are 16 sums over 16 lanes.  Lane j keeps them in an order of its own, sum
+// x in register x ^ j, so that adding them across lanes takes 15 shuffles and additions and no selection, and leaves sum j with
+// lane j: in the step of bit s every lane keeps the registers without the bit and sends the others.
+template <typename T, int RPL>           // state rows of a lane
+__global__ void __launch_bounds__(kThreads, 1) chunk_scan_kernel(const ChunkScanParams cp) {
+    pdl_launch_dependents();
+    constexpr int D = 16 * RPL, C = kChunk;
+    constexpr int STAGE = 3 * C * D + D + 2 * C * C + C + C * 32;       // floats (values: room for fp32)
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    float* stages = reinterpret_cast<float*>(smem_raw);
+    __shared__ float s_read[8][2][C][4];                 // per warp
+    __shared__ __align__(16) float2 s_u[8][C][4];        // (each value twice: a packed pair)
+    const ScanParams& p = cp.s;
+    const int h = blockIdx.y, c0 = blockIdx.x * 32, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, j = lane & 15, grp = lane >> 4;
+    const int d = p.d, dv = p.dv, n = p.M, ncol = min(32, dv - c0);
+    const bool wide_v = dv * (int)sizeof(T) % 16 == 0;
+    for (int i = tid; i < 2 * STAGE; i += kThreads) stages[i] = 0.f;      // rows past the head's width, columns past its values
+    pdl_wait();
+    __syncthreads();
+    auto fetch = [&](int b) {
+        float* st = stages + (b & 1) * STAGE;
+        const int t0 = b * C, nt = min(C, n - t0), t = warp;
+        const size_t row = (size_t)(t0 + t) * p.H + h, ch = (size_t)b * p.H + h;
+        float* at = st + 3 * C * D;
+        float* beta = at + D + 2 * C * C;
+        T* v = reinterpret_cast<T*>(beta + C);
+        if (t < nt) {
+            fetch_row(st + t * D, cp.kt + row * d, d, true, lane);
+            fetch_row(st + (C + t) * D, cp.qt + row * d, d, true, lane);
+            fetch_row(st + (2 * C + t) * D, cp.kh + row * d, d, true, lane);
+            fetch_row(v + t * 32, static_cast<const T*>(p.v) + row * dv + c0, ncol, wide_v, lane);
+            if (lane == 0) cp_async4(smem_u32(beta + t), p.beta + row);
+        } else {
+            for (int c = lane; c < D; c += 32) st[t * D + c] = st[(C + t) * D + c] = st[(2 * C + t) * D + c] = 0.f;
+            if (lane == 0) beta[t] = 0.f;
+        }
+        if (warp == 0) fetch_row(at, cp.decay + ch * d, d, true, lane);
+        if (warp == 1) fetch_row(at + D, cp.coef + ch * 2 * C * C, 2 * C * C, true, lane);
+        asm volatile("cp.async.commit_group;\n" ::: "memory");
+    };
+    fetch(0);
+    // register column c of a lane: column c ^ (j & 1) of its group's two
+    unsigned long long S[RPL / 2][2];                    // rows 64 i + 4 j + (0 .. 3), in pairs
+    const int col = c0 + warp * 4 + grp * 2;
+#pragma unroll
+    for (int i = 0; i < RPL / 4; i++)
+#pragma unroll
+        for (int c = 0; c < 2; c++) {
+            const int r = 64 * i + 4 * j, cc = col + (c ^ (j & 1));
+            float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (r < d && cc < dv) x = *reinterpret_cast<const float4*>(p.state + ((size_t)h * dv + cc) * d + r);
+            S[2 * i][c] = pack2(x.x, x.y);
+            S[2 * i + 1][c] = pack2(x.z, x.w);
+        }
+    const int nb = (n + C - 1) / C, mycol = lane & 3, mytok = lane >> 2;
+    // sum x = 8 (token bit 1) + 4 (token bit 0) + 2 (k or q) + column; where register x of this lane reads
+    int src[4][2];
+#pragma unroll
+    for (int t = 0; t < 4; t++)
+#pragma unroll
+        for (int kind = 0; kind < 2; kind++) src[t][kind] = ((kind ^ ((j >> 1) & 1)) * C + (t ^ (j >> 2))) * D + 4 * j;
+    for (int b = 0; b < nb; b++) {
+        asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+        __syncthreads();                                 // this chunk is here, the one before has been read
+        if (b + 1 < nb) fetch(b + 1);
+        const float* st = stages + (b & 1) * STAGE;
+        const float* at = st + 3 * C * D;
+        const float* beta = at + D + 2 * C * C;
+        const T* v = reinterpret_cast<const T*>(beta + C);
+        // read-outs of the state before the chunk, four tokens at a time
+#pragma unroll
+        for (int t0 = 0; t0 < C; t0 += 4) {
+            float y[16];
+#pragma unroll
+            for (int t = 0; t < 4; t++)
+#pragma unroll
+                for (int kind = 0; kind < 2; kind++) {
+                    unsigned long long a[2] = {0ull, 0ull};
+#pragma unroll
+                    for (int i = 0; i < RPL / 4; i++) {
+                        const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(st + src[t][kind] + t0 * D + 64 * i);
+#pragma unroll
+                        for (int c = 0; c < 2; c++) a[c] = fma2(w.y, S[2 * i + 1][c], fma2(w.x, S[2 * i][c], a[c]));
+                    }
+#pragma unroll
+                    for (int c = 0; c < 2; c++) {
+                        const float2 z = unpack2(a[c]);
+                        y[t * 4 + kind * 2 + c] = z.x + z.y;
+                    }
+                }
+#pragma unroll
+            for (int s = 8; s > 0; s >>= 1)
+#pragma unroll
+                for (int x = 0; x < s; x++) y[x] += __shfl_xor_sync(0xffffffffu, y[x + s], s);
+            s_read[warp][(j >> 1) & 1][t0 + (j >> 2)][grp * 2 + (j & 1)] = y[0];
+        }
+        __syncwarp();
+        // what each token writes: every lane solves its column, and finishes one token's output
+        float u[C];
+#pragma unroll
+        for (int t = 0; t < C; t++) {
+            float r = s_read[warp][0][t][mycol];
+            const float4 a0 = *reinterpret_cast<const float4*>(at + D + t * C), a1 = *reinterpret_cast<const float4*>(at + D + t * C + 4);
+            const float a[C] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
+#pragma unroll
+            for (int i = 0; i < t; i++) r = fmaf(a[i], u[i], r);
+            u[t] = beta[t] * (to_f32<T>(v[t * 32 + warp * 4 + mycol]) - r);
+            if (t == mytok) s_u[warp][t][mycol] = make_float2(u[t], u[t]);
+        }
+        {
+            float o = s_read[warp][1][mytok][mycol];
+            const float4 b0 = *reinterpret_cast<const float4*>(at + D + C * C + mytok * C), b1 = *reinterpret_cast<const float4*>(at + D + C * C + mytok * C + 4);
+            o = fmaf(b0.x, u[0], fmaf(b0.y, u[1], fmaf(b0.z, u[2], fmaf(b0.w, u[3], o))));
+            o = fmaf(b1.x, u[4], fmaf(b1.y, u[5], fmaf(b1.z, u[6], fmaf(b1.w, u[7], o))));
+            const int m = b * C + mytok, cc = c0 + warp * 4 + mycol;
+            if (m < n && cc < dv) p.o[((size_t)m * p.H + h) * dv + cc] = o;
+        }
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < RPL / 4; i++) {
+            const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(at + 64 * i + 4 * j);
+#pragma unroll
+            for (int c = 0; c < 2; c++) {
+                S[2 * i][c] = mul2(w.x, S[2 * i][c]);
+                S[2 * i + 1][c] = mul2(w.y, S[2 * i + 1][c]);
+            }
+        }
+#pragma unroll
+        for (int t = 0; t < C; t++) {
+            unsigned long long u2[2];
+#pragma unroll
+            for (int c = 0; c < 2; c++) u2[c] = *reinterpret_cast<const unsigned long long*>(&s_u[warp][t][grp * 2 + (c ^ (j & 1))]);
+#pragma unroll
+            for (int i = 0; i < RPL / 4; i++) {
+                const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(st + (2 * C + t) * D + 64 * i + 4 * j);
+#pragma unroll
+                for (int c = 0; c < 2; c++) {
+                    S[2 * i][c] = fma2(w.x, u2[c], S[2 * i][c]);
+                    S[2 * i + 1][c] = fma2(w.y, u2[c], S[2 * i + 1][c]);
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < RPL / 4; i++)
+#pragma unroll
+        for (int c = 0; c < 2; c++) {
+            const int r = 64 * i + 4 * j, cc = col + (c ^ (j & 1));
+            const float2 x = unpack2(S[2 * i][c]), y = unpack2(S[2 * i + 1][c]);
+            if (r < d && cc < dv) *reinterpret_cast<float4*>(p.state + ((size_t)h * dv + cc) * d + r) = make_float4(x.x, x.y, y.x, y.y);
+        }
+    roll_inputs<T>(p, n, [](int t) { return t; });
 }
 
 template <int RPL> __host__ __device__ constexpr int scan_block() { return RPL == 32 ? 8 : 16; }      // tokens of a shared-memory block
@@ -318,24 +671,7 @@ __global__ void __launch_bounds__(kThreads) scan_kernel(const ScanParams p) {
             }
         }
     }
-    // the convolutions' last inputs, channels over all CTAs
-    const int prev = p.taps - 1;
-    const T* in = static_cast<const T*>(p.in);
-    T* cs = static_cast<T*>(p.conv_state);
-    if (prev > 0) {
-        for (int c = (blockIdx.y * gridDim.x + blockIdx.x) * kThreads + tid; c < p.channels; c += gridDim.x * gridDim.y * kThreads) {
-            T nv[B200_HYBRID_MAX_TAPS];
-#pragma unroll
-            for (int e = 0; e < B200_HYBRID_MAX_TAPS; e++)
-                if (e < prev) {
-                    const int i = n - prev + e;
-                    nv[e] = i >= 0 ? in[(size_t)row_of(i) * p.pitch + c] : cs[(size_t)(i + prev) * p.pitch + c];
-                }
-#pragma unroll
-            for (int e = 0; e < B200_HYBRID_MAX_TAPS; e++)
-                if (e < prev) cs[(size_t)e * p.pitch + c] = nv[e];
-        }
-    }
+    roll_inputs<T>(p, n, row_of);
 }
 
 template <typename T, int RPL, int MODE>
@@ -361,6 +697,35 @@ void launch_conv_v(const ConvParams& p, bool tree, cudaStream_t st) {
     else launch_kernel(conv_kernel<T, V, NI, false>, dim3(units, (p.M + kConvRows - 1) / kConvRows), dim3(kThreads), 0, st, p);
 }
 
+// Prompts of heads the chunk kernels take.
+bool chunked(const b200_hybrid_layer& l, const b200_hybrid_pass& p) {
+    return !p.tree && p.M > 2 * kChunk && l.dim % 4 == 0 && l.vdim % 4 == 0 && l.dim <= 128 && l.vdim <= 128 && l.conv_taps <= 4;
+}
+
+template <typename T, int RPL>
+int launch_chunk_scan(const ChunkScanParams& p, cudaStream_t st) {
+    constexpr int D = 16 * RPL;
+    const size_t smem = 2 * (size_t)(3 * kChunk * D + D + 2 * kChunk * kChunk + kChunk + kChunk * 32) * 4;
+    launch_kernel(chunk_scan_kernel<T, RPL>, dim3((p.s.dv + 31) / 32, p.s.H), dim3(kThreads), smem, st, p);
+    return check_launch();
+}
+
+template <typename T>
+int delta_chunks(const b200_hybrid_model& m, const b200_hybrid_layer& l, const ConvParams& c, const ScanParams& s, cudaStream_t st) {
+    ChunkParams p{};
+    const size_t nd = (size_t)m.max_rows * l.heads * l.dim, chunks = (m.max_rows + kChunk - 1) / kChunk;
+    p.c = c; p.g = s.g; p.kt = m.chunk; p.qt = m.chunk + nd; p.kh = m.chunk + 2 * nd; p.decay = m.chunk + 3 * nd;
+    p.coef = p.decay + chunks * l.heads * l.dim;
+    const dim3 grid((l.kv_heads + l.heads + 3) / 4, (c.M + kChunk - 1) / kChunk);
+    if (l.conv_taps == 1) launch_kernel(conv_chunk_kernel<T, 1>, grid, dim3(128), 0, st, p);
+    else if (l.conv_taps == 2) launch_kernel(conv_chunk_kernel<T, 2>, grid, dim3(128), 0, st, p);
+    else if (l.conv_taps == 3) launch_kernel(conv_chunk_kernel<T, 3>, grid, dim3(128), 0, st, p);
+    else launch_kernel(conv_chunk_kernel<T, 4>, grid, dim3(128), 0, st, p);
+    if (check_launch() != B200_OK) return B200_ECUDA;
+    const ChunkScanParams q{s, p.kt, p.qt, p.kh, p.decay, p.coef};
+    return l.dim <= 64 ? launch_chunk_scan<T, 4>(q, st) : launch_chunk_scan<T, 8>(q, st);
+}
+
 template <typename T>
 int delta(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_run& r, const b200_hybrid_pass& ps, cudaStream_t st) {
     char* pend = static_cast<char*>(m.pending);
@@ -374,11 +739,6 @@ int delta(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hyb
     c.v = ps.tree ? static_cast<void*>(reinterpret_cast<T*>(pend + r.pend_v) + off * nv) : m.vb;
     c.M = ps.M; c.G = l.kv_heads; c.H = l.heads; c.d = l.dim; c.dv = l.vdim; c.taps = l.conv_taps; c.pitch = delta_pitch(l);
     c.channels = delta_channels(l); c.write_off = ps.write_off;
-    const int most = l.dim > l.vdim ? l.dim : l.vdim;
-    if (l.dim % 4 || l.vdim % 4) launch_conv_v<T, 1, 8>(c, ps.tree, st);
-    else if (most <= 128) launch_conv_v<T, 4, 1>(c, ps.tree, st);
-    else launch_conv_v<T, 4, 2>(c, ps.tree, st);
-    if (check_launch() != B200_OK) return B200_ECUDA;
     ScanParams s{};
     s.q = m.q32; s.state = reinterpret_cast<float*>(cache + r.state_off); s.o = m.o32; s.in = c.in; s.conv_state = cache + r.mix_off;
     s.k = ps.tree ? reinterpret_cast<const float*>(pend + r.pend_k) : m.k32;
@@ -387,7 +747,17 @@ int delta(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hyb
     s.v = ps.tree ? static_cast<const void*>(pend + r.pend_v) : m.vb;
     s.mask = ps.mask; s.M = ps.M; s.H = l.heads; s.G = l.kv_heads; s.d = l.dim; s.dv = l.vdim; s.taps = l.conv_taps; s.pitch = c.pitch;
     s.channels = c.channels;
-    const int rc = ps.tree ? launch_scan<T, kTree>(s, ps.M, st) : launch_scan<T, kChain>(s, 1, st);
+    int rc;
+    if (chunked(l, ps)) {
+        rc = delta_chunks<T>(m, l, c, s, st);
+    } else {
+        const int most = l.dim > l.vdim ? l.dim : l.vdim;
+        if (l.dim % 4 || l.vdim % 4) launch_conv_v<T, 1, 8>(c, ps.tree, st);
+        else if (most <= 128) launch_conv_v<T, 4, 1>(c, ps.tree, st);
+        else launch_conv_v<T, 4, 2>(c, ps.tree, st);
+        if (check_launch() != B200_OK) return B200_ECUDA;
+        rc = ps.tree ? launch_scan<T, kTree>(s, ps.M, st) : launch_scan<T, kChain>(s, 1, st);
+    }
     return rc != B200_OK ? rc : launch_head_norm(m, l, ps.M, m.gb, st);
 }
 
@@ -422,3 +792,9 @@ int launch_delta_commit(const b200_hybrid_model& m, const b200_hybrid_layer& l, 
 
 }  // namespace hybrid
 }  // namespace b200
+
+extern "C" size_t b200_hybrid_chunk_floats(int max_rows, int heads, int dim) {
+    if (max_rows < 1 || heads < 1 || dim < 1) return 0;
+    const size_t nd = (size_t)heads * dim, chunks = ((size_t)max_rows + 7) / 8;
+    return 3 * nd * max_rows + chunks * (nd + (size_t)heads * 128);
+}

@@ -1,6 +1,7 @@
 // Mixture of experts of the hybrid decoders: each row goes through the `top` experts with the largest sigmoid scores of its
 // router logits (fp32), the score multiplies the expert's input.
 //
+//   router_rows                         few rows: logits, a CTA per (expert, row).
 //   expert_up_rows / expert_down_rows   few (row, choice) pairs, or fp32: a warp per channel of a pair; every CTA chooses the
 //                                       row's experts itself from the logits (the choice is a few warp reductions).
 //   route, sort, gather                 many pairs: choices of all rows, their places in expert order (counting sort, a warp
@@ -67,6 +68,21 @@ __device__ __forceinline__ float dot8(const uint4& w, const float* x, float acc)
         acc = fmaf(__uint_as_float(a[i] & 0xffff0000u), b[2 * i + 1], acc);
     }
     return acc;
+}
+
+// Router logits of few rows (many: the matrix product kernels).
+template <typename T>
+__global__ void __launch_bounds__(128) router_rows_kernel(const bf16* w, const T* x, float* z, int experts, int pitch) {
+    pdl_launch_dependents();
+    const int e = blockIdx.x, m = blockIdx.y;
+    __shared__ float red[33];
+    const bf16* wr = w + (size_t)e * pitch;
+    pdl_wait();
+    float a = 0.f;
+#pragma unroll 4
+    for (int k = threadIdx.x * 8; k < pitch; k += 128 * 8) a = dot8(ldg_nc_v4(wr + k), x + (size_t)m * pitch + k, a);
+    a = block_sum(a, red);
+    if (threadIdx.x == 0) z[(size_t)m * experts + e] = a;
 }
 
 struct RowsParams {
@@ -170,20 +186,43 @@ __global__ void __launch_bounds__(kThreads) route_kernel(const float* z, Route r
     }
 }
 
-// One CTA: pairs counted per expert, then placed in expert order, in row order within an expert.
+// One CTA: the pairs' places in expert order, in row order within an expert.  Each warp ranks a run of pairs by itself, then
+// the warps' counts of an expert are added in order.
 __global__ void __launch_bounds__(1024) sort_kernel(Route r, int pairs, int experts) {
     pdl_launch_dependents();
     pdl_wait();
+    extern __shared__ int s_count[];                     // [32][experts], then (expert, rank) of every pair
     __shared__ int s_first[B200_HYBRID_MAX_EXPERTS + 1];
-    extern __shared__ short s_e[];
+    unsigned short* s_e = reinterpret_cast<unsigned short*>(s_count + 32 * experts);
+    unsigned short* s_rank = s_e + pairs;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    for (int e = tid; e <= experts; e += 1024) s_first[e] = 0;
+    const int run = ((pairs + 31) / 32 + 31) / 32 * 32, i0 = warp * run, i1 = min(pairs, i0 + run);
+    for (int i = tid; i < 32 * experts; i += 1024) s_count[i] = 0;
+    for (int i = tid; i < pairs; i += 1024) s_e[i] = (unsigned short)r.expert[i];
     __syncthreads();
-    for (int i = tid; i < pairs; i += 1024) {
-        const int e = r.expert[i];
-        s_e[i] = (short)e;
-        atomicAdd(&s_first[e + 1], 1);
+    int* mine = s_count + warp * experts;
+    for (int i = i0 + lane; i - lane < i1; i += 32) {
+        const int e = i < i1 ? s_e[i] : 0xffff;
+        const unsigned peers = __match_any_sync(0xffffffffu, e);
+        const int before = e != 0xffff ? mine[e] : 0;
+        __syncwarp();
+        if (e != 0xffff) {
+            s_rank[i] = (unsigned short)(before + __popc(peers & ((1u << lane) - 1u)));
+            if (lane == __ffs(peers) - 1) mine[e] = before + __popc(peers);
+        }
+        __syncwarp();
     }
+    __syncthreads();
+    for (int e = tid; e < experts; e += 1024) {
+        int n = 0;
+        for (int w = 0; w < 32; w++) {
+            const int c = s_count[w * experts + e];
+            s_count[w * experts + e] = n;
+            n += c;
+        }
+        s_first[e + 1] = n;
+    }
+    if (tid == 0) s_first[0] = 0;
     __syncthreads();
     if (warp == 0) {
         int before = 0;
@@ -201,20 +240,10 @@ __global__ void __launch_bounds__(1024) sort_kernel(Route r, int pairs, int expe
     }
     __syncthreads();
     for (int e = tid; e <= experts; e += 1024) r.offsets[e] = s_first[e];
-    for (int e = warp; e < experts; e += 32) {
-        int at = s_first[e];
-        if (s_first[e + 1] == at) continue;
-        for (int i0 = 0; i0 < pairs; i0 += 32) {
-            const int i = i0 + lane;
-            const bool hit = i < pairs && s_e[i] == e;
-            const unsigned b = __ballot_sync(0xffffffffu, hit);
-            if (hit) {
-                const int pl = at + __popc(b & ((1u << lane) - 1u));
-                r.place[i] = pl;
-                r.score[pl] = r.raw[i];
-            }
-            at += __popc(b);
-        }
+    for (int i = tid; i < pairs; i += 1024) {
+        const int e = s_e[i], place = s_first[e] + s_count[i / run * experts + e] + s_rank[i];
+        r.place[i] = place;
+        r.score[place] = r.raw[i];
     }
 }
 
@@ -241,9 +270,19 @@ int experts_rows(const b200_hybrid_model& m, const b200_hybrid_layer& l, int row
     return check_launch();
 }
 
-constexpr int kFewPairs = 16;
+constexpr int kFewPairs = 16, kFewRows = 16;
 
 }  // namespace
+
+bool router_in_rows(int rows) { return rows <= kFewRows; }
+
+int launch_router_rows(const b200_hybrid_model& m, const b200_hybrid_layer& l, int rows, cudaStream_t st) {
+    const bf16* w = static_cast<const bf16*>(l.router.w);
+    const dim3 grid(l.experts, rows);
+    if (m.act_type == B200_ACT_F32) launch_kernel(router_rows_kernel<float>, grid, dim3(128), 0, st, w, static_cast<const float*>(m.hb), m.zr, l.experts, l.router.pitch);
+    else launch_kernel(router_rows_kernel<bf16>, grid, dim3(128), 0, st, w, static_cast<const bf16*>(m.hb), m.zr, l.experts, l.router.pitch);
+    return check_launch();
+}
 
 int launch_experts(const b200_hybrid_model& m, const b200_hybrid_layer& l, int rows, const int** place, cudaStream_t st) {
     *place = nullptr;
@@ -252,7 +291,7 @@ int launch_experts(const b200_hybrid_model& m, const b200_hybrid_layer& l, int r
     if (pairs <= kFewPairs) return experts_rows<bf16>(m, l, rows, st);
     const Route r = route_of(m.route, m.max_rows, l.top);
     launch_kernel(route_kernel, dim3((rows + 7) / 8), dim3(kThreads), 0, st, static_cast<const float*>(m.zr), r, rows, l.experts, l.top);
-    const size_t smem = (size_t)pairs * 2;
+    const size_t smem = (size_t)pairs * 4 + (size_t)32 * l.experts * 4;
     if (smem > 200 * 1024) return B200_ELIMIT;
     if (smem > 40 * 1024 && cudaFuncSetAttribute(sort_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return check_launch();
     launch_kernel(sort_kernel, dim3(1), dim3(1024), smem, st, r, pairs, l.experts);

@@ -25,7 +25,7 @@ template <typename T> __device__ __forceinline__ T from_f32(float v);
 template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
 
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float sigmoid_f(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
@@ -84,7 +84,19 @@ enum : int {
     kOpDecay = 7        // exp(-rate softplus(acc + b))
 };
 
-__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// log(1 + e^z) = max(z, 0) + log(1 + x), x = e^-|z| in (0, 1]; log(1 + x) = 2 artanh(s), s = x / (2 + x) <= 1/3, by its odd
+// series up to s^15.
+__device__ __forceinline__ float softplus_f(float z) {
+    const float x = expf(-fabsf(z)), s = __fdividef(x, 2.0f + x), q = s * s;
+    float t = 1.0f / 15.0f;
+    t = fmaf(t, q, 1.0f / 13.0f);
+    t = fmaf(t, q, 1.0f / 11.0f);
+    t = fmaf(t, q, 1.0f / 9.0f);
+    t = fmaf(t, q, 1.0f / 7.0f);
+    t = fmaf(t, q, 1.0f / 5.0f);
+    t = fmaf(t, q, 1.0f / 3.0f);
+    return fmaxf(z, 0.f) + fmaf(2.0f * s * q, t, 2.0f * s);
+}
 
 // Two-branch activations: a product whose columns alternate gate, up, or the same as a kernel of its own.
 struct Gating {
@@ -221,6 +233,7 @@ struct ColumnOut {
         }
 #pragma unroll
         for (int i = 0; i < N; i++) {
+            if (i >= n) break;                       // (n is the same for the whole warp)
             float v = __uint_as_float(acc[i]);
             if (OP == kOpSilu) v = v * sigmoid_f(v);
             else if (OP == kOpSigmoid) v = sigmoid_f(v);
@@ -229,11 +242,9 @@ struct ColumnOut {
             else if (OP == kOpBias) v = v + p0;
             else if (OP == kOpDecay) v = expf(-p1 * softplus_f(v + p0));
             else if (OP == kOpSoftcap) v = p0 > 0.f ? p0 * tanhf(v / p0) : v;
-            if (i < n) {
-                if (F32) *reinterpret_cast<float*>(p + i * stride) = v;
-                else *reinterpret_cast<T*>(p + i * stride) = from_f32<T>(v);
-                if (OP == kOpSoftcap && half_base != nullptr) half_base[(long long)(m0 + i) * (stride >> 2)] = __float2half_rn(v);
-            }
+            if (F32) *reinterpret_cast<float*>(p + i * stride) = v;
+            else *reinterpret_cast<T*>(p + i * stride) = from_f32<T>(v);
+            if (OP == kOpSoftcap && half_base != nullptr) half_base[(long long)(m0 + i) * (stride >> 2)] = __float2half_rn(v);
         }
     }
     // Rows m0 .. m0 + n - 1, n clipped to N: one branch on the operation, straight code for the rows.
@@ -262,9 +273,10 @@ __device__ __forceinline__ void store_gated_rows(const Epi& e, int n, bool valid
     T* dst = static_cast<T*>(e.seg[0].dst) + (n >> 1);
 #pragma unroll
     for (int i = 0; i < N; i += 2) {
+        if (i >= count) break;                       // (the same for the whole warp)
         float a0 = __uint_as_float(acc[i]), a1 = __uint_as_float(acc[i + 1]);
         if (e.row_scale != nullptr) {
-            a0 *= i < count ? e.row_scale[m0 + i] : 0.f;
+            a0 *= e.row_scale[m0 + i];
             a1 *= i + 1 < count ? e.row_scale[m0 + i + 1] : 0.f;
         }
         a0 += b;
@@ -303,7 +315,12 @@ int launch_delta_commit(const b200_hybrid_model& m, const b200_hybrid_layer& l, 
                         const int* rows, int tree_rows, cudaStream_t st);
 // Does the pass read the latent of every head's keys and values written out (prompts), or queries brought into its space?
 bool latent_expands(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_pass& p);
+constexpr int kLatentColumns = 512;      // latent sizes of the bf16 kernel over the latent itself
+int launch_latent_attention(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_run& r, const b200_hybrid_pass& p, cudaStream_t st);
+size_t latent_attention_parts(int rows, int heads);      // partial vectors it may need
 int launch_latent_prep(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hybrid_run& r, const b200_hybrid_pass& p, cudaStream_t st);
+bool router_in_rows(int rows);           // do that few rows get their logits from launch_router_rows?
+int launch_router_rows(const b200_hybrid_model& m, const b200_hybrid_layer& l, int rows, cudaStream_t st);
 // Chooses the experts of every row (router logits in m.zr), runs them and leaves their outputs in rows of m.y; *place: where
 // each (row, choice) is (null: in order).
 int launch_experts(const b200_hybrid_model& m, const b200_hybrid_layer& l, int rows, const int** place, cudaStream_t st);

@@ -3,7 +3,7 @@
 // bf16 activations: one tcgen05 kernel for every row count.  The tile is 128 weight rows (the M of the MMA) x NT token
 // columns; a TMA producer warp streams 128 x 64 weight boxes and NT x 64 activation boxes (128-byte swizzle, K-major)
 // through a shared-memory ring, one thread issues tcgen05.mma (kind::f16, bf16 operands, fp32 accumulator in tensor
-// memory), four warps read the accumulator back (thread = weight row, so stores of neighbouring threads are
+// memory), four or eight warps read the accumulator back (thread = weight row, so stores of neighbouring threads are
 // neighbouring columns of a token's row) and apply the epilogue.  With few tokens a product is a stream of weights:
 // the K range of a tile is then cut over a cluster of up to 8 CTAs whose accumulators are added through distributed
 // shared memory in rank order, so that every SM streams whatever the matrix height.  The weight copies of the first
@@ -26,20 +26,21 @@ namespace {
 constexpr int kTileRows = 128;                    // weight rows of a tile
 constexpr int kTileK = 64;                        // 128 bytes of bf16: one swizzle span
 constexpr int kWBytes = kTileRows * kTileK * 2;
-constexpr int kEpiWarps = 4;
-constexpr int kThreads = (kEpiWarps + 2) * 32;    // + TMA producer warp + MMA warp
 constexpr int kMaxSplit = 8;                      // CTAs of a cluster
 constexpr uint32_t kPolls = 1u << 22;
 constexpr uint32_t kPollNs = 64u;
 
 template <int NT>
 struct Geo {
+    // epilogue warps (a quarter of the tile's rows each; eight: two per quarter, half of the columns each), so that every SM has eight
+    static constexpr int EPI = NT >= 128 ? 8 : 4;
+    static constexpr int THREADS = (EPI + 2) * 32;         // + TMA producer warp + MMA warp
     static constexpr int XBYTES = NT * kTileK * 2;
     static constexpr int STAGE = kWBytes + XBYTES;
-    static constexpr int STAGES = NT == 16 ? 6 : (NT == 32 ? 5 : (NT == 128 ? 6 : 4));
+    static constexpr int STAGES = NT == 16 || NT == 128 ? 6 : (NT == 32 || NT == 160 ? 5 : 4);
     static constexpr int PER_SM = NT <= 64 ? 2 : 1;        // resident CTAs the shared memory allows
     static constexpr int NACC = NT >= 128 ? 2 : 1;
-    static constexpr int ACC_COLS = NT < 32 ? 32 : NT;
+    static constexpr int ACC_COLS = NT < 32 ? 32 : (NT == 160 ? 256 : NT);
     static constexpr int TMEM_COLS = ACC_COLS * NACC;
     static constexpr int SMEM = STAGES * STAGE + 1024 + 256;
 };
@@ -119,8 +120,9 @@ __device__ __forceinline__ float ld_cluster_f32(uint32_t saddr, uint32_t rank) {
 }
 
 template <int NT, bool EXPERTS>
-__global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const __grid_constant__ GemmParams p) {
+__global__ void __launch_bounds__(Geo<NT>::THREADS, Geo<NT>::PER_SM) gemm_kernel(const __grid_constant__ GemmParams p) {
     using G = Geo<NT>;
+    constexpr int kEpiWarps = G::EPI, kThreads = G::THREADS;
     extern __shared__ unsigned char smem_raw[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     uint64_t* bars = reinterpret_cast<uint64_t*>(smem + G::STAGES * G::STAGE);
@@ -277,14 +279,15 @@ __global__ void __launch_bounds__(kThreads, Geo<NT>::PER_SM) gemm_kernel(const _
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
             const Tile at = tile_of(t);
             const int tok0 = at.tok0;
-            const uint32_t taddr = tmem + ab * G::ACC_COLS + ((uint32_t)(warp * 32) << 16);
-            const int r = warp * 32 + lane;
+            const int quarter = warp & 3, cpart = NT * 4 / kEpiWarps, cfirst = (warp >> 2) * cpart;
+            const uint32_t taddr = tmem + ab * G::ACC_COLS + ((uint32_t)(quarter * 32) << 16);
+            const int r = quarter * 32 + lane;
             ColumnOut<bf16> out;
             const bool gated = p.epi.gate.kind != 0;
             if (ks == 1 && !gated) out.init(p.epi, r < at.rows ? at.col0 + r : -1);
             float* part = reinterpret_cast<float*>(smem);          // split: [token][128], over the drained ring
 #pragma unroll 1
-            for (int c = 0; c < NT; c += 16) {
+            for (int c = cfirst; c < cfirst + cpart; c += 16) {
                 if (tok0 + c >= at.tokend) break;
                 uint32_t v[16];
                 asm volatile(
@@ -436,7 +439,7 @@ int launch_gemm(const b200_linear& lin, const void* x, int x_pitch, int x_rows, 
     }
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(grid);
-    cfg.blockDim = dim3(kThreads);
+    cfg.blockDim = dim3(G::THREADS);
     cfg.dynamicSmemBytes = G::SMEM;
     cfg.stream = st;
     cudaLaunchAttribute attrs[2];
@@ -560,7 +563,8 @@ int launch_linear(int act_type, const b200_linear& lin, const void* x, int x_pit
     if (M <= 32) return launch_gemm<32, false>(lin, x, x_pitch, x_rows, epi, M, nullptr, error, st);
     // (few output columns: small token tiles, so that more SMs take part)
     if (M <= 64 || tiles * ((M + 255) / 256) * 2 <= sm_count()) return launch_gemm<64, false>(lin, x, x_pitch, x_rows, epi, M, nullptr, error, st);
-    if (M <= 128) return launch_gemm<128, false>(lin, x, x_pitch, x_rows, epi, M, nullptr, error, st);
+    // (short K: a tile's epilogue is most of its time, and smaller tiles even out over the SMs)
+    if (M <= 128 || lin.pitch <= 512) return launch_gemm<128, false>(lin, x, x_pitch, x_rows, epi, M, nullptr, error, st);
     return launch_gemm<256, false>(lin, x, x_pitch, x_rows, epi, M, nullptr, error, st);
 }
 
@@ -568,10 +572,13 @@ int launch_linear_experts(const b200_linear& lin, const void* x, int x_rows, int
     if (!lin.w || !x || !offsets || lin.n < 1 || lin.pitch < 64 || lin.pitch % 64 != 0 || rows < 1 || x_rows < rows) return B200_EINVAL;
     if (lin.groups < 1 || lin.groups > B200_HYBRID_MAX_EXPERTS) return B200_ELIMIT;
     if (!aligned16(lin.w) || !aligned16(x)) return B200_EALIGN;
+    // One token tile for most experts, with room for an uneven load: a second tile streams an expert's weights again.
     const int mean = rows / lin.groups;
-    if (mean <= 24) return launch_gemm<32, true>(lin, x, lin.pitch, x_rows, epi, rows, offsets, error, st);
-    if (mean <= 80) return launch_gemm<64, true>(lin, x, lin.pitch, x_rows, epi, rows, offsets, error, st);
-    return launch_gemm<128, true>(lin, x, lin.pitch, x_rows, epi, rows, offsets, error, st);
+    if (mean <= 20) return launch_gemm<32, true>(lin, x, lin.pitch, x_rows, epi, rows, offsets, error, st);
+    if (mean <= 48) return launch_gemm<64, true>(lin, x, lin.pitch, x_rows, epi, rows, offsets, error, st);
+    if (mean <= 100) return launch_gemm<128, true>(lin, x, lin.pitch, x_rows, epi, rows, offsets, error, st);
+    if (mean <= 140) return launch_gemm<160, true>(lin, x, lin.pitch, x_rows, epi, rows, offsets, error, st);
+    return launch_gemm<256, true>(lin, x, lin.pitch, x_rows, epi, rows, offsets, error, st);
 }
 
 }  // namespace hybrid

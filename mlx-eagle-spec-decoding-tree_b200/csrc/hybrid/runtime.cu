@@ -1,6 +1,8 @@
 // The pass driver: walks the layer runs and issues their launches; C entry points of libb200hybrid.so.
 #include "hybrid.cuh"
 
+#include <limits.h>
+
 namespace b200 {
 int g_last_cuda_error = 0;
 int g_use_pdl = 1;
@@ -169,7 +171,8 @@ int feed_forward(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b
     const int pitch = round_up(l.ff, 64);
     if (l.ff_kind == B200_FF_EXPERTS) {
         const int* place = nullptr;
-        B200_TRY(product(m, p, l.router, m.hb, one_seg(plain_seg(0, l.experts, kOpNone, 1, m.zr, l.experts)), p.M, st));
+        if (router_in_rows(p.M)) B200_TRY(launch_router_rows(m, l, p.M, st));
+        else B200_TRY(product(m, p, l.router, m.hb, one_seg(plain_seg(0, l.experts, kOpNone, 1, m.zr, l.experts)), p.M, st));
         B200_TRY(launch_experts(m, l, p.M, &place, st));
         return launch_join(m, m.norm_out ? l.norm2 : nullptr, p.M, l.top, place, inject, st);
     }
@@ -216,9 +219,9 @@ bool valid(const b200_hybrid_model& m, const b200_hybrid_pass& p) {
             if (!l.gate_bias || !l.gate_lower || !l.head_norm) return false;
         } else if (l.mixer == B200_MIXER_DELTA) {
             if (l.kv_heads < 1 || l.heads % l.kv_heads || l.conv_taps < 1 || l.conv_taps > B200_HYBRID_MAX_TAPS || l.low_rank < 1) return false;
-            if (!l.mix_conv || !l.decay_bias || !l.decay_rate || !l.head_norm || !m.cb || !m.lowb || !m.q32 || !m.k32 || !m.beta) return false;
+            if (!l.mix_conv || !l.decay_bias || !l.decay_rate || !l.head_norm || !m.cb || !m.lowb || !m.q32 || !m.k32 || !m.beta || !m.chunk) return false;
         } else if (l.mixer == B200_MIXER_LATENT) {
-            if (l.kv_rank < 1 || l.rot_dim < 2 || l.rot_dim % 2 || l.maps != 1 || l.window < 1 || l.keep_first < 0) return false;
+            if (l.kv_rank < 1 || l.rot_dim < 2 || l.rot_dim % 2 || l.maps != 1 || l.window != INT_MAX || l.keep_first != 0) return false;
             if (!l.rot_freq || !l.latent_norm || !m.lat32 || !m.qn || !m.ob || !m.attn_part) return false;
         } else {
             return false;

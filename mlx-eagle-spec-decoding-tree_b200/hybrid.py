@@ -631,6 +631,9 @@ class HybridModel:
         experts = [l for l in self.layers if l.ff_kind == FF_EXPERTS]
         top, n_exp = max([l.top for l in experts], default=0), max([l.experts for l in experts], default=0)
         self.route = torch.zeros(max(_lib.hybrid().b200_hybrid_route_ints(R, top, n_exp), 4), dtype=torch.int32, device=dev)
+        deltas = [l for l in self.layers if l.mixer == MIXER_DELTA]
+        chunk = max([_lib.hybrid().b200_hybrid_chunk_floats(R, l.heads, l.dim) for l in deltas], default=0)
+        self.chunk = torch.zeros(max(chunk, 4), dtype=f32, device=dev)
         self.expanded: List[torch.Tensor] = []
         self.tok_buf = torch.zeros(R, dtype=torch.int32, device=dev)
         self.pos_buf = torch.zeros(R, dtype=torch.int32, device=dev)
@@ -649,6 +652,7 @@ class HybridModel:
         for k, t in b.items():
             setattr(d, k, t.data_ptr() if t is not None else None)
         d.route, d.route_top, d.route_experts = self.route.data_ptr(), top, n_exp
+        d.chunk = self.chunk.data_ptr()
         d.error = self.error.data_ptr()
         self._desc = d
         self.pending = torch.zeros(max(self.cache_layout(64).pending_bytes, ALIGN), dtype=torch.uint8, device=dev)
