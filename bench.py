@@ -23,7 +23,7 @@ length 0 and above: random-init pairs accept nothing, so the headline counts one
 Other workloads: ``c2`` draft-only tree build (0.5B-shape draft, prompt 128, depth 3, 7 nodes), ``c4``
 Llama-3-8B-shape target + Llama-3.2-1B-shape draft (prompt 1024, depth 4, 31 verify tokens, also reports the
 time to the first token of the 1024-token prompt), ``tp70b`` / ``tp7b`` one stream with the target cut across
-all ranks, ``hybrid`` the layer-list design beside the 4-bit models of equal size (plain decoding, prompts).  ``--impl reference`` times the CPU restatement only (the reference itself is MLX/Metal and cannot
+all ranks, ``hybrid`` the layer-list designs beside the 4-bit models of equal size (plain decoding, prompts).  ``--impl reference`` times the CPU restatement only (the reference itself is MLX/Metal and cannot
 run on Linux), on the same configuration, and prints the same line with ``"impl": "reference"``.
 """
 from __future__ import annotations
@@ -727,8 +727,21 @@ def batched_requests_numbers(torch, be, base, draft, depth, verify, prompt_len, 
     return out
 
 
-# layer-list design beside the 4-bit model of the same width, feed-forward and layer count
-HYBRID_PAIRS = {"1b": ("zaverax-1b", "llama3.2-1b"), "8b": ("zaverax-8b", "llama3-8b")}
+# layer-list designs beside the 4-bit model of the same width, feed-forward weights per token and layer count
+HYBRID_PAIRS = {"1b": ("zaverax-1b", "zokelix-1b", "llama3.2-1b"), "8b": ("zaverax-8b", "zokelix-8b", "llama3-8b")}
+
+
+def cache_bytes_read(args, prompt_len):
+    """Bytes of K/V rows one token of a layer-list model reads at a context of ``prompt_len`` (bf16 cache)."""
+    n = 0
+    for li, _ in args.runs:
+        sp = args.layers[li]
+        mx = sp.mixer
+        if sp.type == "attention":
+            n += 2 * min(prompt_len, mx["mask"]["size"]) * mx["kv_heads"] * (2 * mx["dim"] + mx["vdim"])
+        elif sp.type == "latent_attention":
+            n += 2 * prompt_len * (mx["kv_rank"] + mx["rot_dim"])
+    return n
 
 
 def hybrid_numbers(torch, be, name, dev, prompt_len, steps, layers=0):
@@ -742,20 +755,14 @@ def hybrid_numbers(torch, be, name, dev, prompt_len, steps, layers=0):
     if os.path.exists(mpath):
         with open(mpath) as f:
             tensor_peak = float(json.load(f).get("bf16_tflops", tensor_peak))
-    if name.startswith("zaverax"):
+    listed = name.split("-")[0] in ("zaverax", "zokelix")
+    if listed:
         args = be.HybridArgs.from_config(be.hybrid.preset_config(name))
         if layers:
             args = dataclasses.replace(args, layers=args.layers[:layers])
         m = be.HybridModel.random_init(args, 7, dev, max_rows=max(256, prompt_len))
         state = m.cache_layout(64).state_bytes
-        kv = 0
-        for li, _ in args.runs:
-            sp = args.layers[li]
-            if sp.type == "attention":
-                mx = sp.mixer
-                keys = min(prompt_len, mx["mask"]["size"])
-                kv += 2 * keys * mx["kv_heads"] * (2 * mx["dim"] + mx["vdim"])
-        stream = m.linear_weight_bytes() + kv + 2 * state              # the states are read and written
+        stream = m.linear_weight_bytes() + cache_bytes_read(m.args, prompt_len) + 2 * state      # the states are read and written
         macs = m.linear_weight_bytes() // 2
         head = args.vocab_size * args.width
     else:
@@ -802,7 +809,7 @@ def hybrid_numbers(torch, be, name, dev, prompt_len, steps, layers=0):
 
     t_step = timed(decode, 5) / steps
     m.check_fused_error()
-    out = {"model": name, "layers": m.args.num_hidden_layers, "weights": "bf16" if name.startswith("zaverax") else "4 bit",
+    out = {"model": name, "layers": m.args.num_hidden_layers, "weights": "bf16" if listed else "4 bit",
            "decode_tokens_per_s": round(1 / t_step, 1), "decode_ms": round(t_step * 1e3, 4), "decode_bytes": stream,
            "decode_frac_of_hbm": round(stream / t_step / 1e9 / peak, 3), "prompt_tokens": prompt_len,
            "prompt_tokens_per_s": round(prompt_len / t_prompt), "prompt_ms": round(t_prompt * 1e3, 3),
@@ -813,8 +820,8 @@ def hybrid_numbers(torch, be, name, dev, prompt_len, steps, layers=0):
 
 
 def run_hybrid(args, torch, be, dev, local_rank):
-    """``--workload hybrid``: the layer-list design at two sizes beside the 4-bit model of equal size (plain decoding
-    at the prompt's context length, prompt ingestion); one JSON line, ``value`` = decoded tokens/s of the 8b-size design."""
+    """``--workload hybrid``: the layer-list designs at two sizes beside each other and the 4-bit model of equal size (plain
+    decoding at the prompt's context length, prompt ingestion); one JSON line, ``value`` = decoded tokens/s of zaverax-8b."""
     steps = args.steps
     if args.hybrid_model:
         print(json.dumps(hybrid_numbers(torch, be, args.hybrid_model, dev, 1024, steps, args.layers)))
@@ -864,7 +871,7 @@ def main():
     ap.add_argument("--workload", default="c3", choices=["streams", "hybrid"] + sorted(STREAM_WORKLOADS) + sorted(TP_WORKLOADS),
                     help="c3 (= streams, the default): one independent request stream per GPU; c2: draft-only tree build; c4: "
                          "Llama-3-8B/3.2-1B shapes, prompt 1024; tp70b / tp7b: one stream with the target cut across all ranks; hybrid: "
-                         "the layer-list design beside the 4-bit models of equal size (one GPU)")
+                         "the layer-list designs beside the 4-bit models of equal size (one GPU)")
     args = ap.parse_args()
     if args.workload == "streams":
         args.workload = "c3"

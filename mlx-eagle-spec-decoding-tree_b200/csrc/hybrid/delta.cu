@@ -10,6 +10,7 @@
 //                    chain   the pass's rows in order; the new state and convolution inputs are written back;
 //                    tree    a CTA per row replays the row's path from the state, nothing is written back;
 //                    commit  pending rows are replayed and written back, no output.
+//   step_kernel    one token: convolution, unit norms, the step of the state, head norm and output gate, a CTA per head.
 //   conv_chunk_kernel, chunk_scan_kernel
 //                  prompts: 8 tokens at a time.  With P_j the product of the chunk's decays up to token j and P_ij that of the
 //                  tokens after i up to j (products of decays only, nothing is divided),
@@ -697,6 +698,153 @@ void launch_conv_v(const ConvParams& p, bool tree, cudaStream_t st) {
     else launch_kernel(conv_kernel<T, V, NI, false>, dim3(units, (p.M + kConvRows - 1) / kConvRows), dim3(kThreads), 0, st, p);
 }
 
+// ---------------------------------------------------------------- one token
+struct StepParams {
+    const void* in;          // [pitch] convolution inputs of the token
+    void* conv_state;        // [taps - 1][pitch]
+    const float* w;          // [taps][channels]
+    const float* g;          // [H * d]
+    const float* beta;       // [H]
+    float* state;            // [H][dv][d]
+    const float* norm;       // [dv]
+    const void* gate;        // [H * dv]
+    void* out;               // [H * dv]
+    int H, G, d, dv, taps, pitch, channels;
+    float eps;
+};
+
+// CTA = head; the heads of one key head form a cluster, so that the convolution inputs they share move on after all have read
+// them.  8 lanes per state column hold its rows; heads of at most 128 x 128, multiples of 4.
+template <typename T>
+__global__ void __launch_bounds__(kThreads) step_kernel(const StepParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    constexpr int IT = 4, MAX = 128;
+    __shared__ __align__(16) float sq[MAX], sk[MAX], sg[MAX], sv[MAX], so[MAX];
+    __shared__ float red[33];
+    const int h = blockIdx.x, R = p.H / p.G, kh = h / R, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, j = lane & 7, d = p.d, dv = p.dv;
+    float4 S[IT][4];                                     // rows 32 i + 4 j + (0 .. 3) of column 32 it + 4 warp + lane / 8
+    float* sbase = p.state + (size_t)h * dv * d;
+#pragma unroll
+    for (int it = 0; it < IT; it++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int col = 32 * it + 4 * warp + (lane >> 3), r = 32 * i + 4 * j;
+            S[it][i] = col < dv && r < d ? *reinterpret_cast<const float4*>(sbase + (size_t)col * d + r) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    const T* in = static_cast<const T*>(p.in);
+    T* cs = static_cast<T*>(p.conv_state);
+    if (tid < MAX) {
+        sg[tid] = tid < d ? p.g[(size_t)h * d + tid] : 0.f;
+        sq[tid] = sk[tid] = sv[tid] = 0.f;
+    }
+    __syncthreads();
+    T moved[2][B200_HYBRID_MAX_TAPS];                    // the channel's inputs after the token
+    int chan[2];
+#pragma unroll
+    for (int x = 0; x < 2; x++) {
+        const int e = tid + x * kThreads, which = e / MAX, c = e % MAX;
+        const bool mine = which < 3 && c < (which == 2 ? dv : d);
+        chan[x] = !mine ? -1 : (which == 2 ? 2 * p.G * d + h * dv + c : (which * p.G + kh) * d + c);
+        if (!mine) continue;
+        float z = 0.f;
+#pragma unroll
+        for (int t = 0; t < B200_HYBRID_MAX_TAPS; t++) {
+            if (t >= p.taps) break;
+            moved[x][t] = t == p.taps - 1 ? in[chan[x]] : cs[(size_t)t * p.pitch + chan[x]];
+            z = fmaf(p.w[(size_t)t * p.channels + chan[x]], to_f32<T>(moved[x][t]), z);
+        }
+        z *= sigmoid_f(z);
+        (which == 0 ? sq : (which == 1 ? sk : sv))[c] = which == 2 ? to_f32<T>(from_f32<T>(z)) : z;
+    }
+    if (R > 1) asm volatile("barrier.cluster.arrive.release.aligned;\nbarrier.cluster.wait.acquire.aligned;\n" ::: "memory");
+#pragma unroll
+    for (int x = 0; x < 2; x++) {
+        const bool key = tid + x * kThreads < 2 * MAX;   // (the key head's inputs move once)
+        if (chan[x] < 0 || (key && h % R != 0)) continue;
+#pragma unroll
+        for (int t = 1; t < B200_HYBRID_MAX_TAPS; t++)
+            if (t < p.taps) cs[(size_t)(t - 1) * p.pitch + chan[x]] = moved[x][t];
+    }
+    __syncthreads();
+    if (warp < 2) {
+        float* v = warp == 0 ? sq : sk;
+        float4 x = *reinterpret_cast<const float4*>(v + 4 * lane);
+        const float f = rsqrtf(warp_sum(x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w) + 1e-6f) * (warp == 0 ? rsqrtf((float)d) : 1.f);
+        *reinterpret_cast<float4*>(v + 4 * lane) = make_float4(x.x * f, x.y * f, x.z * f, x.w * f);
+    }
+    __syncthreads();
+    const float beta = p.beta[h];
+    float ss = 0.f;
+#pragma unroll
+    for (int it = 0; it < IT; it++) {
+        const int col = 32 * it + 4 * warp + (lane >> 3);
+        if (32 * it >= dv) break;
+        float r = 0.f, o = 0.f;
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const float4 g = *reinterpret_cast<const float4*>(sg + 32 * i + 4 * j), k = *reinterpret_cast<const float4*>(sk + 32 * i + 4 * j);
+            float4& s = S[it][i];
+            s = make_float4(s.x * g.x, s.y * g.y, s.z * g.z, s.w * g.w);
+            r = fmaf(k.x, s.x, fmaf(k.y, s.y, fmaf(k.z, s.z, fmaf(k.w, s.w, r))));
+        }
+#pragma unroll
+        for (int x = 1; x < 8; x <<= 1) r += __shfl_xor_sync(0xffffffffu, r, x);
+        const float u = beta * (sv[min(col, MAX - 1)] - r);
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const float4 q = *reinterpret_cast<const float4*>(sq + 32 * i + 4 * j), k = *reinterpret_cast<const float4*>(sk + 32 * i + 4 * j);
+            float4& s = S[it][i];
+            s = make_float4(fmaf(k.x, u, s.x), fmaf(k.y, u, s.y), fmaf(k.z, u, s.z), fmaf(k.w, u, s.w));
+            o = fmaf(q.x, s.x, fmaf(q.y, s.y, fmaf(q.z, s.z, fmaf(q.w, s.w, o))));
+            const int row = 32 * i + 4 * j;
+            if (col < dv && row < d) *reinterpret_cast<float4*>(sbase + (size_t)col * d + row) = s;
+        }
+#pragma unroll
+        for (int x = 1; x < 8; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
+        if (j == 0 && col < dv) {
+            so[col] = o;
+            ss = fmaf(o, o, ss);
+        }
+    }
+    const float rstd = rsqrtf(block_sum(ss, red) / (float)dv + p.eps);
+    for (int c = tid; c < dv; c += kThreads)
+        static_cast<T*>(p.out)[(size_t)h * dv + c] = from_f32<T>(so[c] * rstd * p.norm[c] * to_f32<T>(static_cast<const T*>(p.gate)[(size_t)h * dv + c]));
+}
+
+// Single tokens that step_kernel takes.
+bool single_step(const b200_hybrid_layer& l, const b200_hybrid_pass& p) {
+    return !p.tree && p.M == 1 && l.dim % 4 == 0 && l.vdim % 4 == 0 && l.dim <= 128 && l.vdim <= 128 && l.heads / l.kv_heads <= 8;
+}
+
+template <typename T>
+int delta_step(const b200_hybrid_model& m, const b200_hybrid_layer& l, const ScanParams& s, const float* w, cudaStream_t st) {
+    StepParams p{};
+    p.in = s.in; p.conv_state = s.conv_state; p.w = w; p.g = s.g; p.beta = s.beta; p.state = s.state; p.norm = l.head_norm; p.gate = m.gb;
+    p.out = m.ab; p.H = s.H; p.G = s.G; p.d = s.d; p.dv = s.dv; p.taps = s.taps; p.pitch = s.pitch; p.channels = s.channels; p.eps = m.eps;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(p.H);
+    cfg.blockDim = dim3(kThreads);
+    cfg.stream = st;
+    cudaLaunchAttribute attrs[2];
+    int na = 0;
+    if (p.H > p.G) {
+        attrs[na].id = cudaLaunchAttributeClusterDimension;
+        attrs[na].val.clusterDim.x = p.H / p.G;
+        attrs[na].val.clusterDim.y = attrs[na].val.clusterDim.z = 1;
+        na++;
+    }
+    if (g_use_pdl) {
+        attrs[na].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attrs[na].val.programmaticStreamSerializationAllowed = 1;
+        na++;
+    }
+    cfg.attrs = attrs;
+    cfg.numAttrs = na;
+    cudaLaunchKernelEx(&cfg, step_kernel<T>, p);
+    return check_launch();
+}
+
 // Prompts of heads the chunk kernels take.
 bool chunked(const b200_hybrid_layer& l, const b200_hybrid_pass& p) {
     return !p.tree && p.M > 2 * kChunk && l.dim % 4 == 0 && l.vdim % 4 == 0 && l.dim <= 128 && l.vdim <= 128 && l.conv_taps <= 4;
@@ -747,6 +895,7 @@ int delta(const b200_hybrid_model& m, const b200_hybrid_layer& l, const b200_hyb
     s.v = ps.tree ? static_cast<const void*>(pend + r.pend_v) : m.vb;
     s.mask = ps.mask; s.M = ps.M; s.H = l.heads; s.G = l.kv_heads; s.d = l.dim; s.dv = l.vdim; s.taps = l.conv_taps; s.pitch = c.pitch;
     s.channels = c.channels;
+    if (single_step(l, ps)) return delta_step<T>(m, l, s, l.mix_conv, st);
     int rc;
     if (chunked(l, ps)) {
         rc = delta_chunks<T>(m, l, c, s, st);

@@ -239,7 +239,7 @@ using namespace b200::hybrid;
 
 extern "C" {
 
-int b200_hybrid_version(void) { return 1; }
+int b200_hybrid_version(void) { return 2; }
 int b200_hybrid_last_cuda_error(void) { return g_last_cuda_error; }
 void b200_hybrid_set_pdl(int enabled) { g_use_pdl = enabled ? 1 : 0; }
 

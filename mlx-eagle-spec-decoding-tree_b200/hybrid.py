@@ -219,7 +219,7 @@ class GatedRecurrence(Mixer):
 class ChannelDelta(Mixer):
     """Gated delta rule with a decay per key channel; short convolutions on queries, keys and values; low-rank decay and
     output gate (their ranks are given by the tensors)."""
-    launches = 6                 # projections, low-rank products, convolutions, scan, head norm, output product
+    launches = 4                 # projections, low-rank products, step, output product (decoding)
 
     @staticmethod
     def ranks(mx: dict) -> tuple:

@@ -69,6 +69,16 @@ def test_delta_ranks_come_from_the_tensors(be, cuda, ranks):
         check(be, cfg, 60, dtype, [[60], [1]], w=w)
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_decays_of_every_size(be, cuda, dtype):
+    """Channels that keep everything, lose everything at once, and all between."""
+    cfg = hc.zokelix([hc.delta(heads=2, kv_heads=1, dim=32, vdim=20)])
+    w = hc.weights(cfg, 4)
+    w["l0.mix.dt_bias"] = torch.linspace(-25.0, 25.0, 64).bfloat16()
+    w["l0.mix.A_log"] = torch.tensor([-2.0, 1.5]).bfloat16()
+    check(be, cfg, 120, dtype, [[120], [1], [19, 40, 3]], w=w)
+
+
 LATENT = {
     "plain": dict(),
     "unscaled": dict(scaling=None),
@@ -80,6 +90,7 @@ LATENT = {
     "real_sizes": dict(heads=2, dim=128, rot_dim=64, vdim=128, kv_rank=512),
     "past_the_prompt_kernel": dict(heads=2, dim=250, rot_dim=20, vdim=136, kv_rank=72),
     "sharp": dict(scale=1.1),
+    "middle_rank": dict(heads=6, dim=20, rot_dim=18, vdim=70, kv_rank=200),
 }
 
 
@@ -114,7 +125,7 @@ def test_gated_feed_forward(be, cuda, ff, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("mlp", [hc.moe(), hc.moe(1, 1, 30), hc.moe(2, 2, 9), hc.moe(16, 1, 33), hc.moe(40, 6, 65, 0.3), hc.moe(35, 10, 20, 100.0),
-                                 hc.moe(3, 1, 300, 0.7)], ids=lambda m: "{experts}of{top}".format(**m["router"]))
+                                 hc.moe(3, 1, 300, 0.7), hc.moe(3, 2, 50)], ids=lambda m: "{experts}of{top}".format(**m["router"]))
 def test_experts(be, cuda, mlp, dtype):
     cfg = hc.zokelix([hc.delta(mlp=mlp)], width=120)
     w = hc.weights(cfg, mlp["expert"]["ff"])
