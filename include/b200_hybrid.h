@@ -69,7 +69,7 @@ typedef struct b200_hybrid_layer {
     int low_rank;                       /* columns of the low-rank inputs of decay and output gate together          */
     const float* mix_conv;              /* [conv_taps][2*kv_heads*dim + heads*vdim], last tap: the current token     */
     const float* decay_bias;            /* [heads*dim]                                                               */
-    const float* decay_rate;            /* [heads*dim]: g = exp(-rate * softplus(z + bias))                          */
+    const float* decay_rate;            /* [heads*dim]: g = exp(-rate * softplus(z + bias)); kept as g - 1            */
     b200_linear low;                    /* rows decay | output gate over the low-rank inputs                         */
     /* latent */
     int kv_rank, rot_dim;

@@ -501,6 +501,9 @@ template <typename T, int QN>
 int launch_rows_shared(AttnParams& p, cudaStream_t st) {
     if (p.vdim <= 2 * kRowThreads) return launch_rows_c<T, QN, 2, true>(p, st);
     if (p.vdim <= 4 * kRowThreads) return launch_rows_c<T, QN, 4, true>(p, st);
+    if constexpr (QN <= 8) {
+        if (p.vdim <= 8 * kRowThreads) return launch_rows_c<T, QN, 8, true>(p, st);
+    }
     return B200_ELIMIT;
 }
 
@@ -538,10 +541,11 @@ int launch_prompt_any(const AttnParams& p, cudaStream_t st) {
     return launch_prompt<8, MAPS, LATENT>(p, st);
 }
 
-// Few-row passes of a latent layer: all heads read the same rows.  Heads of a CTA: what the shared memory holds.
+// Passes of a latent layer that walk the latent itself, other than latent.cu's: all heads read the same rows.  Heads of a CTA:
+// what the shared memory holds.
 int launch_latent_rows(const b200_hybrid_model& m, const b200_hybrid_layer& l, AttnParams& p, int max_keys, cudaStream_t st) {
     const int elem = act_bytes(m.act_type);
-    int most = 16;
+    int most = p.vdim <= 4 * kRowThreads ? 16 : 8;
     while (most > 4 && rows_smem(p, most, elem, true) > kMaxSmem) most /= 2;
     p.qgroups = (p.H + most - 1) / most;
     p.hpg = (p.H + p.qgroups - 1) / p.qgroups;

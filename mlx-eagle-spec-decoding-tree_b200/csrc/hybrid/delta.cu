@@ -1,7 +1,9 @@
 // Gated delta rule of the hybrid decoders, one decay per head and key channel:
 //     S <- g * S (rows);   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q,
 // q and k unit vectors; q, k, v come out of short causal convolutions with silu.  Everything that enters the recurrence is
-// fp32, the state [heads][vdim][dim] is carried in the request's cache, as are the convolutions' last inputs.
+// fp32, the state [heads][vdim][dim] is carried in the request's cache, as are the convolutions' last inputs.  Decays are kept
+// as g - 1 and applied as S <- S + (g - 1) S: a decay next to 1, rounded, would change a state by as much as it loses over
+// thousands of tokens.
 //
 //   conv_kernel    convolution, silu and unit norm: a warp per head of q, k or v and block of rows.
 //   scan_kernel    token by token.  CTA = (head, 32 state columns); 8 lanes share a column and hold its rows in registers (packed
@@ -165,11 +167,11 @@ __device__ __forceinline__ float transpose_sum32(float (&v)[32], int lane) {
 
 struct ChunkParams {
     ConvParams c;            // (q, k unused)
-    const float* g;          // [M][H * d]
+    const float* g;          // [M][H * d], decays - 1
     float* kt;               // [M][H * d]: P_j k_j
     float* qt;               // P_j q_j
     float* kh;               // P_j7 k_j
-    float* decay;            // [chunks][H * d]: P_7
+    float* decay;            // [chunks][H * d]: P_7 - 1
     float* coef;             // [chunks][H][2][8][8]: k_j . P_ij k_i (i < j), q_j . P_ij k_i (i <= j), zeros elsewhere
 };
 
@@ -254,19 +256,19 @@ __global__ void __launch_bounds__(128) conv_chunk_kernel(const ChunkParams p) {
         float g[kChunk][4];
 #pragma unroll
         for (int r = 0; r < kChunk; r++) {
-            float4 x = make_float4(1.f, 1.f, 1.f, 1.f);
+            float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
             if (in && r < rows) x = *reinterpret_cast<const float4*>(p.g + ((size_t)(r0 + r) * H + h) * d + c);
             g[r][0] = x.x; g[r][1] = x.y; g[r][2] = x.z; g[r][3] = x.w;
         }
-        float P[4] = {1.f, 1.f, 1.f, 1.f};
+        float P[4] = {0.f, 0.f, 0.f, 0.f};                   // products - 1: (1 + a)(1 + b) - 1 = a + b + ab
 #pragma unroll
         for (int r = 0; r < kChunk; r++) {
 #pragma unroll
-            for (int e = 0; e < 4; e++) P[e] *= g[r][e];
+            for (int e = 0; e < 4; e++) P[e] = fmaf(P[e], g[r][e], P[e] + g[r][e]);
             if (in && r < rows) {
                 const size_t at = ((size_t)(r0 + r) * H + h) * d + c;
-                *reinterpret_cast<float4*>(p.kt + at) = make_float4(P[0] * k[r][0], P[1] * k[r][1], P[2] * k[r][2], P[3] * k[r][3]);
-                *reinterpret_cast<float4*>(p.qt + at) = make_float4(P[0] * q[r][0], P[1] * q[r][1], P[2] * q[r][2], P[3] * q[r][3]);
+                *reinterpret_cast<float4*>(p.kt + at) = make_float4(fmaf(P[0], k[r][0], k[r][0]), fmaf(P[1], k[r][1], k[r][1]), fmaf(P[2], k[r][2], k[r][2]), fmaf(P[3], k[r][3], k[r][3]));
+                *reinterpret_cast<float4*>(p.qt + at) = make_float4(fmaf(P[0], q[r][0], q[r][0]), fmaf(P[1], q[r][1], q[r][1]), fmaf(P[2], q[r][2], q[r][2]), fmaf(P[3], q[r][3], q[r][3]));
             }
         }
         if (in) *reinterpret_cast<float4*>(p.decay + ((size_t)chunk * H + h) * d + c) = make_float4(P[0], P[1], P[2], P[3]);
@@ -296,7 +298,7 @@ __global__ void __launch_bounds__(128) conv_chunk_kernel(const ChunkParams p) {
             for (int j = i; j < kChunk; j++) {
                 if (j > i)
 #pragma unroll
-                    for (int e = 0; e < 4; e++) w[e] *= g[j][e];
+                    for (int e = 0; e < 4; e++) w[e] = fmaf(w[e], g[j][e], w[e]);
                 qd[j] = w[0] * q[j][0] + w[1] * q[j][1] + w[2] * q[j][2] + w[3] * q[j][3];
                 if (j > i) put(w[0] * k[j][0] + w[1] * k[j][1] + w[2] * k[j][2] + w[3] * k[j][3]);
             }
@@ -310,7 +312,7 @@ __global__ void __launch_bounds__(128) conv_chunk_kernel(const ChunkParams p) {
 struct ScanParams {
     const float* q;          // [M][G * d]
     const float* k;          // chain: [M][G * d]; tree, commit: pending rows
-    const float* g;          // [..][H * d]
+    const float* g;          // [..][H * d], decays - 1
     const float* beta;       // [..][H]
     const void* v;           // [..][H * dv]
     float* state;            // [H][dv][d]
@@ -495,8 +497,8 @@ __global__ void __launch_bounds__(kThreads, 1) chunk_scan_kernel(const ChunkScan
             const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(at + 64 * i + 4 * j);
 #pragma unroll
             for (int c = 0; c < 2; c++) {
-                S[2 * i][c] = mul2(w.x, S[2 * i][c]);
-                S[2 * i + 1][c] = mul2(w.y, S[2 * i + 1][c]);
+                S[2 * i][c] = fma2(w.x, S[2 * i][c], S[2 * i][c]);
+                S[2 * i + 1][c] = fma2(w.y, S[2 * i + 1][c], S[2 * i + 1][c]);
             }
         }
 #pragma unroll
@@ -618,8 +620,8 @@ __global__ void __launch_bounds__(kThreads) scan_kernel(const ScanParams p) {
                     const ulonglong2 g = g4[8 * i], k = k4[8 * i];
                     k2[2 * i] = k.x;
                     k2[2 * i + 1] = k.y;
-                    S[2 * i] = mul2(S[2 * i], g.x);
-                    S[2 * i + 1] = mul2(S[2 * i + 1], g.y);
+                    S[2 * i] = fma2(S[2 * i], g.x, S[2 * i]);
+                    S[2 * i + 1] = fma2(S[2 * i + 1], g.y, S[2 * i + 1]);
                     a0 = fma2(k.x, S[2 * i], a0);
                     a1 = fma2(k.y, S[2 * i + 1], a1);
                 }
@@ -703,7 +705,7 @@ struct StepParams {
     const void* in;          // [pitch] convolution inputs of the token
     void* conv_state;        // [taps - 1][pitch]
     const float* w;          // [taps][channels]
-    const float* g;          // [H * d]
+    const float* g;          // [H * d], decays - 1
     const float* beta;       // [H]
     float* state;            // [H][dv][d]
     const float* norm;       // [dv]
@@ -785,7 +787,7 @@ __global__ void __launch_bounds__(kThreads) step_kernel(const StepParams p) {
         for (int i = 0; i < 4; i++) {
             const float4 g = *reinterpret_cast<const float4*>(sg + 32 * i + 4 * j), k = *reinterpret_cast<const float4*>(sk + 32 * i + 4 * j);
             float4& s = S[it][i];
-            s = make_float4(s.x * g.x, s.y * g.y, s.z * g.z, s.w * g.w);
+            s = make_float4(fmaf(s.x, g.x, s.x), fmaf(s.y, g.y, s.y), fmaf(s.z, g.z, s.z), fmaf(s.w, g.w, s.w));
             r = fmaf(k.x, s.x, fmaf(k.y, s.y, fmaf(k.z, s.z, fmaf(k.w, s.w, r))));
         }
 #pragma unroll

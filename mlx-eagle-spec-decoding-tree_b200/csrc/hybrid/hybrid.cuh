@@ -81,7 +81,7 @@ enum : int {
     kOpResidual = 4,    // dst += mult * (acc + b) (+ add), b optional
     kOpSoftcap = 5,     // cap * tanh(acc / cap), cap <= 0: acc
     kOpBias = 6,        // acc + b
-    kOpDecay = 7        // exp(-rate softplus(acc + b))
+    kOpDecay = 7        // exp(-rate softplus(acc + b)) - 1: what is lost keeps its precision where almost nothing is
 };
 
 // log(1 + e^z) = max(z, 0) + log(1 + x), x = e^-|z| in (0, 1]; log(1 + x) = 2 artanh(s), s = x / (2 + x) <= 1/3, by its odd
@@ -196,7 +196,7 @@ struct ColumnOut {
         if (op == kOpForget) return (1.0f - p1) * sigmoid_f(-(acc + p0));
         if (op == kOpResidual) return residual + p0 * (acc + bias);
         if (op == kOpBias) return acc + p0;
-        if (op == kOpDecay) return expf(-p1 * softplus_f(acc + p0));
+        if (op == kOpDecay) return expm1f(-p1 * softplus_f(acc + p0));
         if (op == kOpSoftcap && p0 > 0.f) return p0 * tanhf(acc / p0);
         return acc;
     }
@@ -240,7 +240,7 @@ struct ColumnOut {
             else if (OP == kOpForget) v = (1.0f - p1) * sigmoid_f(-(v + p0));
             else if (OP == kOpResidual) v = r[i] + p0 * (v + bias);
             else if (OP == kOpBias) v = v + p0;
-            else if (OP == kOpDecay) v = expf(-p1 * softplus_f(v + p0));
+            else if (OP == kOpDecay) v = expm1f(-p1 * softplus_f(v + p0));
             else if (OP == kOpSoftcap) v = p0 > 0.f ? p0 * tanhf(v / p0) : v;
             if (F32) *reinterpret_cast<float*>(p + i * stride) = v;
             else *reinterpret_cast<T*>(p + i * stride) = from_f32<T>(v);

@@ -90,7 +90,7 @@ struct RowsParams {
     const int* pos;
     const unsigned long long* mask;
     const int* prefix;
-    int M, H, cp, width, rank, rows, tree, tail, splits, out_pitch;
+    int M, H, cp, width, rows, tree, tail, splits, out_pitch;
     float scale_log2;
 
     // Cache rows of the pass: committed ones, then its own (chain) or the tail.
@@ -306,7 +306,7 @@ int launch_latent_attention(const b200_hybrid_model& m, const b200_hybrid_layer&
     p.width = latent_pitch(l);
     p.q = static_cast<const bf16*>(m.qb); p.cache = reinterpret_cast<const bf16*>(static_cast<const char*>(ps.cache) + r.k_off);
     p.part = m.attn_part; p.out = static_cast<bf16*>(m.ob); p.pos = ps.pos; p.mask = ps.mask; p.prefix = ps.prefix;
-    p.M = ps.M; p.H = l.heads; p.rank = l.kv_rank; p.rows = ps.cache_rows; p.tree = ps.tree; p.tail = ps.tree ? ps.tail : 0;
+    p.M = ps.M; p.H = l.heads; p.rows = ps.cache_rows; p.tree = ps.tree; p.tail = ps.tree ? ps.tail : 0;
     p.out_pitch = l.value.pitch; p.scale_log2 = l.scale * kLog2e;
     const int keys = ps.max_keys + p.tail, groups = (p.M * p.H + kVecs - 1) / kVecs;
     p.splits = splits_for(groups, ((keys < ps.cache_rows ? keys : ps.cache_rows) + kBlock - 1) / kBlock);

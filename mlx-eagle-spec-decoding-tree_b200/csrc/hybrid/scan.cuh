@@ -23,12 +23,6 @@ __device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigne
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
     return r;
 }
-__device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigned long long b) {
-    unsigned long long r;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-    return r;
-}
-
 // One row of `n` elements to shared memory by a warp: 16-byte asynchronous copies where the row allows them.
 template <typename E>
 __device__ __forceinline__ void fetch_row(E* dst, const E* src, int n, bool wide, int lane) {

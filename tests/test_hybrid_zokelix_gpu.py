@@ -79,6 +79,19 @@ def test_decays_of_every_size(be, cuda, dtype):
     check(be, cfg, 120, dtype, [[120], [1], [19, 40, 3]], w=w)
 
 
+def test_decays_next_to_one_keep_their_precision(be, cuda):
+    """Hundreds of tokens at decays of 1 - 1e-5: a decay rounded to fp32 would be off by up to 3e-8 every time."""
+    cfg = hc.zokelix([hc.delta(heads=2, kv_heads=2, dim=16, vdim=16)])
+    w, toks = hc.weights(cfg, 5), hc.tokens(cfg, 700, 5)
+    for n in ("a1", "a2"):
+        w[f"l0.mix.{n}"].zero_()
+    w["l0.mix.dt_bias"].fill_(-11.5)
+    w["l0.mix.b"][:, :] = 0
+    ref, _ = oracle(cfg, w, toks)
+    for cuts in ([700], [3, 1]):
+        assert errors(feed(build(be, cfg, w, "float32"), toks, cuts), ref).max() < 4e-6
+
+
 LATENT = {
     "plain": dict(),
     "unscaled": dict(scaling=None),
@@ -90,6 +103,7 @@ LATENT = {
     "real_sizes": dict(heads=2, dim=128, rot_dim=64, vdim=128, kv_rank=512),
     "past_the_prompt_kernel": dict(heads=2, dim=250, rot_dim=20, vdim=136, kv_rank=72),
     "sharp": dict(scale=1.1),
+    "wide_latent": dict(heads=9, dim=20, rot_dim=14, vdim=30, kv_rank=600),
     "middle_rank": dict(heads=6, dim=20, rot_dim=18, vdim=70, kv_rank=200),
 }
 
